@@ -602,6 +602,66 @@ int nvllm_embedding_stream(float* h, void* x, int32_t x_dtype, const void* table
 int nvllm_moe_route_logits(int32_t* topk_idx, float* topk_w, const float* logits, int64_t ld, const float* bias, int32_t n,
                            int32_t experts, int32_t top, void* stream);
 
+/* ---- Norm after the sum, weighted head norms before the rotation, kept first keys, per-head delta rule, gated linear
+ * attention, the clamped gate in the GEMM epilogue ---------------------------------------------------------------------- */
+
+/* h = rms(alpha * h + y) * w;   out = last_w ? rms(h) * last_w : h.   h: f32 [n, hidden], updated in place; y in y_dtype, out
+ * in out_dtype; weights f32 (last_w nullable: the model's last norm behind the last layer).  hidden <= 49152. */
+int nvllm_rms_sum_norm(void* out, float* h, const void* y, int32_t y_dtype, float alpha, const float* w, const float* last_w,
+                       int32_t n, int32_t hidden, float eps, int32_t out_dtype, void* stream);
+/* nvllm_rope_table_interleaved with wavelength-dependent scaling of the frequencies f_i = base^(-2i/dims), off for factor <= 0:
+ * with l = 2 pi / f:  l < original / high: f;   l > original / low: f / factor;   between: (1 - s) f / factor + s f with
+ * s = (original / l - low) / (high - low). */
+int nvllm_rope_table_scaled(float* cos_sin, int32_t max_pos, int32_t dims, double base, double factor, double low, double high,
+                            double original, void* stream);
+/* Attention preparation with a weighted RMS norm per query and key head (weights f32 [dim], shared by the heads, nullable: 1)
+ * BEFORE the rotation of the head's first rot_dims values (pairing as in nvllm_attn_rotary_store).  proj: f32 rows
+ * [q (heads x dim) | k (kv_heads x dim) | v (kv_heads x vdim) | ...].  q in `dtype`, k / v into cache rows slots[i] (slot < 0:
+ * nothing stored).  v_first (f32 [n, kv_heads * vdim], rows ldvf apart, nullable) without v_lambda: also receives the values;
+ * with v_lambda (one f32 on the device): the stored value is (1 - lambda) v + lambda v_first. */
+int nvllm_attn_norm_rotary_store(void* q, int64_t ldq, void* k_cache, void* v_cache, int64_t k_row, int64_t v_row, const float* proj,
+                                 int64_t ldp, const float* q_norm_w, const float* k_norm_w, float norm_eps,
+                                 const int64_t* positions, const float* rope_table, int32_t rot_dims, int32_t halves,
+                                 int32_t max_pos, float* v_first, int64_t ldvf, const float* v_lambda, const int32_t* slots,
+                                 int32_t n, int32_t heads, int32_t kv_heads, int32_t dim, int32_t vdim, int32_t dtype, void* stream);
+/* nvllm_biased_attention with keep_first > 0: the keys 0 .. keep_first - 1 (as far as they are not in the future) stay visible
+ * outside the window or chunk. */
+int nvllm_masked_attention(void* out, int64_t ldo, const void* q, int64_t ldq, const float* gate, int64_t ldg,
+                           int32_t gate_per_head, const void* k_cache, const void* v_cache, int64_t k_row, int64_t v_row,
+                           const int32_t* tok_seq, const int64_t* positions, const int32_t* block_tables, int32_t table_cap,
+                           int32_t block_size, int32_t n, int32_t heads, int32_t kv_heads, int32_t dim, int32_t vdim, float scale,
+                           float softcap, float temp_coef, int32_t temp_every, int32_t window, int32_t keep_first,
+                           const float* sinks, int32_t chunk, const float* head_scale, const float* dist_bias, int32_t dist_rows,
+                           const float* out_rot_table, int32_t max_pos, const int32_t* cu_tokens, int32_t n_seqs, int32_t dtype,
+                           void* stream);
+/* nvllm_delta_prepare / nvllm_gated_delta_recurrence with ONE decay per head: decay [n, heads] (rows ldd apart), dt_bias [heads];
+ * S <- g_t S with g_t a number. */
+int nvllm_head_delta_prepare(float* q, int64_t ldq, float* k, int64_t ldk, float* beta, int64_t ldb, float* decay, int64_t ldd,
+                             const float* a_log, const float* dt_bias, int32_t n, int32_t heads, int32_t groups, int32_t dk,
+                             float q_scale, float unit_eps, void* stream);
+int nvllm_head_delta_recurrence(float* y, int64_t ldy, const float* q, int64_t ldq, const float* k, int64_t ldk, const float* v,
+                                int64_t ldv, const float* decay, int64_t ldd, const float* beta, int64_t ldb, float* state,
+                                const int32_t* seq_slot, const int32_t* cu_tokens, const int64_t* positions, int32_t n_seqs,
+                                int32_t heads, int32_t groups, int32_t dk, int32_t dv, void* stream);
+/* Gated linear attention (sequence / slot conventions of nvllm_linear_recurrence): per head S <- diag(decay_t) S + k_t v_t^T,
+ * y_t = q_scale S^T q_t.  decay: f32 [n, heads * dk], rows ldd apart.  dk <= 512. */
+int nvllm_channel_recurrence(float* y, int64_t ldy, const float* q, int64_t ldq, const float* k, int64_t ldk, const float* v,
+                             int64_t ldv, const float* decay, int64_t ldd, float q_scale, float* state, const int32_t* seq_slot,
+                             const int32_t* cu_tokens, const int64_t* positions, int32_t n_seqs, int32_t heads, int32_t groups,
+                             int32_t dk, int32_t dv, void* stream);
+/* out[t, c] = sigmoid(sum_r x[t, r] w2[r, c] + bias[c])^(1 / tau): the second step of a two-step decay projection, all f32;
+ * w2: [rank, channels] (the projection's weight transposed), bias nullable. */
+int nvllm_low_rank_decay(float* out, int64_t ldo, const float* x, int64_t ldx, const float* w2, const float* bias, int32_t n,
+                         int32_t rank, int32_t channels, float tau, void* stream);
+/* nvllm_gemm_silu_mul_bf16 with the gate as a parameter: limit > 0: y = g' sigmoid(1.702 g') (u' + 1) with g' = min(gate, limit),
+ * u' = up clamped to [-limit, limit] (as nvllm_glu_clamped); limit <= 0: SiLU. */
+int nvllm_gemm_glu_bf16(void* out, const void* x, const void* w_gate_up, int32_t m, int32_t inter, int32_t k, int64_t ldx,
+                        int64_t ldw, int64_t ldout, float limit, void* workspace, size_t workspace_bytes, void* stream);
+/* The same over expert groups (128-row tiles, tile_group as in nvllm_gemm_bf16_grouped): w holds per group [gate (inter rows) |
+ * up (inter rows)] x k, y is [max_rows, inter].  inter % 64 == 0. */
+int nvllm_gemm_glu_bf16_grouped(void* y, const void* x, const void* w, int32_t max_rows, int32_t inter, int32_t k, int32_t groups,
+                                int64_t ldx, int64_t ldw, int64_t ldy, const int32_t* tile_group, float limit, void* stream);
+
 /* ------------------------------------------------------------------------------------------------
  * Engine-level C ABI: the C++ host runtime that mirrors the reference's Rust types one-to-one
  * (Config, SamplingParams, Sequence, BlockManager, Scheduler, ModelRunner, Qwen3Model, LLMEngine).

@@ -126,6 +126,19 @@ PROTOTYPES = {
     "nvllm_gated_delta_recurrence": (i32, [vp, i64, vp, i64, vp, i64, vp, i64, vp, i64, vp, i64, vp, vp, vp, vp, i32, i32, i32, i32, i32,
                                            vp]),
     "nvllm_gated_group_norm_act": (i32, [vp, i64, vp, i64, vp, i64, vp, i32, i32, i32, i32, f32, i32, i32, i32, vp]),
+    "nvllm_rms_sum_norm": (i32, [vp, vp, vp, i32, f32, vp, vp, i32, i32, f32, i32, vp]),
+    "nvllm_rope_table_scaled": (i32, [vp, i32, i32, f64, f64, f64, f64, f64, vp]),
+    "nvllm_attn_norm_rotary_store": (i32, [vp, i64, vp, vp, i64, i64, vp, i64, vp, vp, f32, vp, vp, i32, i32, i32, vp, i64, vp, vp, i32, i32,
+                                           i32, i32, i32, i32, vp]),
+    "nvllm_masked_attention": (i32, [vp, i64, vp, i64, vp, i64, i32, vp, vp, i64, i64, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32,
+                                     f32, f32, f32, i32, i32, i32, vp, i32, vp, vp, i32, vp, i32, vp, i32, i32, vp]),
+    "nvllm_head_delta_prepare": (i32, [vp, i64, vp, i64, vp, i64, vp, i64, vp, vp, i32, i32, i32, i32, f32, f32, vp]),
+    "nvllm_head_delta_recurrence": (i32, [vp, i64, vp, i64, vp, i64, vp, i64, vp, i64, vp, i64, vp, vp, vp, vp, i32, i32, i32, i32, i32,
+                                          vp]),
+    "nvllm_channel_recurrence": (i32, [vp, i64, vp, i64, vp, i64, vp, i64, vp, i64, f32, vp, vp, vp, vp, i32, i32, i32, i32, i32, vp]),
+    "nvllm_low_rank_decay": (i32, [vp, i64, vp, i64, vp, vp, i32, i32, i32, f32, vp]),
+    "nvllm_gemm_glu_bf16": (i32, [vp, vp, vp, i32, i32, i32, i64, i64, i64, f32, vp, sz, vp]),
+    "nvllm_gemm_glu_bf16_grouped": (i32, [vp, vp, vp, i32, i32, i32, i32, i64, i64, i64, vp, f32, vp]),
 }
 
 

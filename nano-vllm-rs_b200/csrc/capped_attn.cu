@@ -4,6 +4,7 @@
 //   * an optional output gate:   out *= sigmoid(gate)       (gate: f32 pre-activations, same layout as the output),
 //   * key and value sizes that may differ (dim, vdim),
 //   * an optional sliding window: position p sees the keys p - window + 1 .. p   (window <= 0: all keys 0 .. p),
+//     and, with keep > 0, the first `keep` keys of its sequence whatever their distance,
 //   * optional sinks: a learned number per head whose exponential joins the softmax denominator (no key, no value),
 //   * the gate as one number per head instead of one per output value.
 // Every query token carries its sequence (a row of the block tables) and its position, so one launch serves whole prompts,
@@ -12,6 +13,7 @@
 // nvllm_attn_bias_store: the step before it — adds the projection biases, writes the queries in the operand type and the
 // keys / values into their cache rows.  nvllm_attn_rope_norm_store: the same step for layers with rotary positions on pairs
 // of neighbouring dimensions, a weightless per-head RMS norm after the rotation, and values that are the un-rotated keys.
+// nvllm_attn_norm_rotary_store: a weighted per-head RMS norm before the rotation, values mixed with an earlier layer's.
 // Scores, softmax and the accumulation of P.V are f32.
 #include "common.cuh"
 
@@ -291,6 +293,147 @@ __global__ void __launch_bounds__(128) attn_rotary_store_halves_vec_kernel(const
   }
 }
 
+// The step for layers that norm every query and key head (with a weight shared by the heads) BEFORE the rotation, and whose
+// values may be mixed with those of an earlier layer:
+//   head -> rms(head) * w (w: [dim]), then the rotation of its first rot_dims values; a value head -> its cache row, where
+//   v_first != null and lambda == null: the values also go to v_first (f32, [n, kv_heads * vdim]), for later layers;
+//   v_first and lambda: what is stored is (1 - lambda) v + lambda v_first, lambda one number on the device.
+struct NormStoreArgs {
+  void* q; int64_t ldq;
+  void *kc, *vc; int64_t k_row, v_row;
+  const float* proj; int64_t ldp;
+  const float *qw, *kw; float eps;
+  const int64_t* positions; const float2* table; int rot_dims, halves, max_pos;
+  float* v_first; int64_t ldvf; const float* lambda;
+  const int32_t* slots;
+  int n, heads, kv_heads, dim, vdim;
+};
+
+// One warp per (token, head) over the heads [q heads | key heads | value heads]; any sizes, both pairings.
+template <typename T>
+__global__ void __launch_bounds__(128) attn_norm_rotary_store_kernel(const NormStoreArgs a) {
+  const int lane = threadIdx.x & 31, per = a.heads + 2 * a.kv_heads;
+  const int64_t item = static_cast<int64_t>(blockIdx.x) * 4 + (threadIdx.x >> 5);
+  if (item >= static_cast<int64_t>(a.n) * per) return;
+  const int t = static_cast<int>(item / per), hh = static_cast<int>(item % per);
+  const int32_t slot = a.slots[t];
+  const bool is_q = hh < a.heads, is_v = hh >= a.heads + a.kv_heads;
+  if (!is_q && slot < 0) return;
+  const float* p = a.proj + static_cast<int64_t>(t) * a.ldp;
+  const int qn = a.heads * a.dim, kn = a.kv_heads * a.dim;
+  if (is_v) {
+    const int g = hh - a.heads - a.kv_heads;
+    const float* src = p + qn + kn + static_cast<int64_t>(g) * a.vdim;
+    float* vf = a.v_first ? a.v_first + t * a.ldvf + static_cast<int64_t>(g) * a.vdim : nullptr;
+    T* dst = static_cast<T*>(a.vc) + slot * a.v_row + static_cast<int64_t>(g) * a.vdim;
+    const float lam = a.lambda ? *a.lambda : 0.f;
+    for (int c = lane; c < a.vdim; c += 32) {
+      float v = src[c];
+      if (a.lambda) v = (1.0f - lam) * v + lam * vf[c];
+      else if (vf) vf[c] = v;
+      stv(dst + c, v);
+    }
+    return;
+  }
+  const int h = is_q ? hh : hh - a.heads;
+  const float* src = p + (is_q ? 0 : qn) + static_cast<int64_t>(h) * a.dim;
+  const float* w = is_q ? a.qw : a.kw;
+  float sq = 0.f;
+  for (int c = lane; c < a.dim; c += 32) sq = fmaf(src[c], src[c], sq);
+  const float r = 1.0f / sqrtf(warp_sum(sq) / a.dim + a.eps);
+  int64_t pos = a.positions[t];
+  pos = pos < 0 ? 0 : (pos >= a.max_pos ? a.max_pos - 1 : pos);
+  const int hr = a.rot_dims / 2;
+  const float2* tab = a.table + pos * hr;
+  T* dst = is_q ? static_cast<T*>(a.q) + t * a.ldq + static_cast<int64_t>(h) * a.dim
+                : static_cast<T*>(a.kc) + slot * a.k_row + static_cast<int64_t>(h) * a.dim;
+  for (int c = lane; c < a.dim; c += 32) {
+    float v = src[c] * r * (w ? w[c] : 1.0f);
+    if (c < a.rot_dims) {
+      const int pc = a.halves ? (c < hr ? c + hr : c - hr) : (c ^ 1);
+      const bool second = a.halves ? c >= hr : (c & 1);
+      const float o = src[pc] * r * (w ? w[pc] : 1.0f);
+      const float2 cs = tab[a.halves ? (c < hr ? c : c - hr) : (c >> 1)];
+      v = second ? fmaf(v, cs.x, o * cs.y) : fmaf(v, cs.x, -o * cs.y);   // (u cos - v sin, v cos + u sin)
+    }
+    stv(dst + c, v);
+  }
+}
+
+// The halves pairing with 16-byte accesses: dim, vdim multiples of 4 up to 512, rot_dims a multiple of 8, aligned rows.  The
+// head stays in registers; a chunk's partner in the rotation is read again (it is in L1).
+template <typename T>
+__global__ void __launch_bounds__(128) attn_norm_rotary_store_vec_kernel(const NormStoreArgs a) {
+  const int lane = threadIdx.x & 31, per = a.heads + 2 * a.kv_heads;
+  const int64_t item = static_cast<int64_t>(blockIdx.x) * 4 + (threadIdx.x >> 5);
+  if (item >= static_cast<int64_t>(a.n) * per) return;
+  const int t = static_cast<int>(item / per), hh = static_cast<int>(item % per);
+  const int32_t slot = a.slots[t];
+  const bool is_q = hh < a.heads, is_v = hh >= a.heads + a.kv_heads;
+  if (!is_q && slot < 0) return;
+  const int h = is_q ? hh : (is_v ? hh - a.heads - a.kv_heads : hh - a.heads);
+  const int qn = a.heads * a.dim, kn = a.kv_heads * a.dim, size = is_v ? a.vdim : a.dim, nv = size / 4;
+  const float4* src = reinterpret_cast<const float4*>(a.proj + static_cast<int64_t>(t) * a.ldp + (is_q ? 0 : (is_v ? qn + kn : qn)) +
+                                                      static_cast<int64_t>(h) * size);
+  T* dst = is_q ? static_cast<T*>(a.q) + t * a.ldq + static_cast<int64_t>(h) * size
+                : (is_v ? static_cast<T*>(a.vc) + slot * a.v_row : static_cast<T*>(a.kc) + slot * a.k_row) + static_cast<int64_t>(h) * size;
+  auto put = [&](int c, const float4& o) {
+    if (sizeof(T) == 2) *reinterpret_cast<uint2*>(dst + 4 * c) = make_uint2(pack_bf16x2(o.x, o.y), pack_bf16x2(o.z, o.w));
+    else *reinterpret_cast<float4*>(dst + 4 * c) = o;
+  };
+  if (is_v) {
+    float4* vf = a.v_first ? reinterpret_cast<float4*>(a.v_first + t * a.ldvf + static_cast<int64_t>(h) * size) : nullptr;
+    const float lam = a.lambda ? *a.lambda : 0.f, own = 1.0f - lam;
+    for (int c = lane; c < nv; c += 32) {
+      float4 x = src[c];
+      if (a.lambda) {
+        const float4 f = vf[c];
+        x = make_float4(own * x.x + lam * f.x, own * x.y + lam * f.y, own * x.z + lam * f.z, own * x.w + lam * f.w);
+      } else if (vf) {
+        vf[c] = x;
+      }
+      put(c, x);
+    }
+    return;
+  }
+  const float4* w = reinterpret_cast<const float4*>(is_q ? a.qw : a.kw);
+  int64_t pos = a.positions[t];
+  pos = pos < 0 ? 0 : (pos >= a.max_pos ? a.max_pos - 1 : pos);
+  const float4* tab = reinterpret_cast<const float4*>(a.table + pos * (a.rot_dims / 2));   // (cos, sin) of two pairs per float4
+  float4 v[4];
+  float sq = 0.f;
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    const int c = lane + 32 * k;
+    if (c < nv) {
+      v[k] = src[c];
+      sq += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+    }
+  }
+  const float r = 1.0f / sqrtf(warp_sum(sq) / size + a.eps);
+  const int hr4 = a.rot_dims / 8;   // chunks in half the rotated part
+  auto normed = [&](const float4& x, int c) {
+    const float4 ww = w ? w[c] : make_float4(1.f, 1.f, 1.f, 1.f);
+    return make_float4(x.x * r * ww.x, x.y * r * ww.y, x.z * r * ww.z, x.w * r * ww.w);
+  };
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    const int c = lane + 32 * k;
+    if (c < nv) {
+      float4 x = normed(v[k], c);
+      if (c < 2 * hr4) {
+        const bool second = c >= hr4;
+        const int pc = second ? c - hr4 : c + hr4, m = second ? c - hr4 : c;
+        const float4 o = normed(src[pc], pc), cs0 = tab[2 * m], cs1 = tab[2 * m + 1];
+        const float sg = second ? 1.0f : -1.0f;                 // (u cos - v sin, v cos + u sin)
+        x.x = fmaf(x.x, cs0.x, sg * o.x * cs0.y); x.y = fmaf(x.y, cs0.z, sg * o.y * cs0.w);
+        x.z = fmaf(x.z, cs1.x, sg * o.z * cs1.y); x.w = fmaf(x.w, cs1.z, sg * o.w * cs1.w);
+      }
+      put(c, x);
+    }
+  }
+}
+
 struct AttnArgs {
   void* out; int64_t ldo;
   const void* q; int64_t ldq;
@@ -302,6 +445,7 @@ struct AttnArgs {
   int window; const float* sinks; int gate_per_head;
   const int32_t* dense_cu;   // non-null (and tables null): keys are not paged, key j of sequence s is row dense_cu[s] + j
   // positional options of nvllm_biased_attention (all off when zero / null)
+  int keep;                  // > 0: the keys 0 .. keep - 1 stay visible outside the window (or chunk), at their true positions
   int chunk;                 // > 0: position p sees only the keys of its own chunk, floor(p / chunk) * chunk .. p
   const float* head_scale;   // [heads]: a factor per head on the scaled score
   const float* dist_bias;    // [heads, dist_rows]: added to the score of key j: dist_bias[h, min(p - j, dist_rows - 1)]
@@ -349,11 +493,12 @@ __global__ void __launch_bounds__(128) capped_attn_warp_kernel(const AttnArgs a)
   for (int i = 0; i < kMaxVPerLane; ++i) acc[i] = 0.f;
   const int nkeys = static_cast<int>(pos) + 1;
   const int first = first_key(a, static_cast<int>(pos));   // passes start at multiples of 32 whatever the window or chunk
-  for (int j0 = first & ~31; j0 < nkeys; j0 += 32) {
+  for (int j0 = a.keep > 0 ? 0 : first & ~31; j0 < nkeys; j0 += 32) {
+    if (j0 >= a.keep && j0 < (first & ~31)) j0 = first & ~31;   // past the kept keys: on to the window
     const int j = j0 + lane;
     float s = -INFINITY;
     int64_t slot = -1;
-    if (j < nkeys && j >= first) {
+    if (j < nkeys && (j >= first || j < a.keep)) {
       const int32_t blk = table ? table[j / a.block_size] : 0;
       if (blk >= 0) {
         slot = table ? static_cast<int64_t>(blk) * a.block_size + j % a.block_size : dense0 + j;
@@ -452,7 +597,7 @@ __device__ __forceinline__ float fast_tanh(float x) { return 1.0f - __fdividef(2
 template <int DMAX, int VMAX, int NP, int VP, int QS, int VS, bool EXT>
 __device__ __forceinline__ void attn_tile(float (&o)[VMAX / 8][4], float (&m)[2], float (&l)[2], uint32_t q_addr, uint32_t k_addr,
                                           uint32_t v_addr, int key0, const int (&pos)[2], const int (&lo)[2], const float (&qscale)[2],
-                                          bool capped, float cap2, bool need_mask, int tq4, const float* const (&bias)[2], int dist_rows) {
+                                          bool capped, float cap2, bool need_mask, int tq4, const float* const (&bias)[2], int dist_rows, int keep) {
   float s[2 * NP][4];
 #pragma unroll
   for (int i = 0; i < 2 * NP; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
@@ -477,7 +622,7 @@ __device__ __forceinline__ void attn_tile(float (&o)[VMAX / 8][4], float (&m)[2]
       float v = s[nt][e] * qscale[i];            // with a cap: the score over the cap; without: the score in log2 units
       if (capped) v = cap2 * fast_tanh(v);
       if (EXT) { if (bias[i] != nullptr && j <= pos[i]) v = fmaf(bias[i][min(pos[i] - j, dist_rows - 1)], kLog2e, v); }
-      if (need_mask) v = (j <= pos[i] && j >= lo[i]) ? v : -INFINITY;   // lo: the first key of the row's window or chunk
+      if (need_mask) v = (j <= pos[i] && (j >= lo[i] || j < keep)) ? v : -INFINITY;   // lo: the first key of the row's window or chunk
       s[nt][e] = v;
       mx[i] = fmaxf(mx[i], v);
     }
@@ -576,10 +721,11 @@ __global__ void __launch_bounds__(kThreads, 2) capped_attn_mma_kernel(const Attn
   };
   // thread -> (key row, every fourth 16-byte chunk of it): no index arithmetic in the copy loop
   const int lr = tid >> 2, lh = tid & 3;
-  auto load_tile = [&](int kt, int buf) {
+  auto load_tile = [&](int it) {
+    const int buf = it & 1;
     bf16* kd = Ks + buf * kKeys * QS + lr * QS;
     bf16* vd = Vs + buf * kKeys * VS + lr * VS;
-    const int64_t slot = slot_s[kt & 1][lr];
+    const int64_t slot = slot_s[buf][lr];
     const bf16* ksrc = slot >= 0 ? kc + slot * a.k_row : kc;
     const bf16* vsrc = slot >= 0 ? vc + slot * a.v_row : vc;
     const int nb = slot >= 0 ? 16 : 0;
@@ -622,34 +768,39 @@ __global__ void __launch_bounds__(kThreads, 2) capped_attn_mma_kernel(const Attn
   // with a window the first tile is the one that holds the first key the CTA's first token sees (tiles stay anchored at
   // multiples of 64 from the sequence's start)
   const int kt0 = first_key(a, static_cast<int>(a.positions[tok0])) / kKeys;   // (windows and chunks only move forward with the position)
-  if (tid < kKeys) { slot_s[kt0 & 1][tid] = lookup(kt0); slot_s[(kt0 + 1) & 1][tid] = lookup(kt0 + 1); }
+  // the tiles of the kept first keys come before the window's; tile number `it` of the walk is key tile tile_of(it)
+  const int nkeep = min((a.keep + kKeys - 1) / kKeys, kt0), iters = nkeep + ntiles - kt0;
+  auto tile_of = [&](int it) { return it < nkeep ? it : it - nkeep + kt0; };
+  if (tid < kKeys) { slot_s[0][tid] = lookup(tile_of(0)); slot_s[1][tid] = lookup(tile_of(1)); }
   __syncthreads();
-  load_tile(kt0, kt0 & 1);
+  load_tile(0);
   const uint32_t q_addr = smem_u32(Qs + (rbase + (lane & 15)) * QS + (lane >> 4) * 8);
   const int k_lane = ((lane & 7) + (lane >> 4) * 8) * QS + ((lane >> 3) & 1) * 8;
   const int v_lane = ((lane & 7) + ((lane >> 3) & 1) * 8) * VS + (lane >> 4) * 8;
-  for (int kt = kt0; kt < ntiles; ++kt) {
-    const int buf = kt & 1;
-    if (kt + 1 < ntiles) { load_tile(kt + 1, buf ^ 1); cp_async_wait<1>(); } else { cp_async_wait<0>(); }
-    const int64_t slot_ahead = (tid < kKeys && kt + 2 < ntiles) ? lookup(kt + 2) : -1;   // in flight during this tile's math
+  for (int it = 0; it < iters; ++it) {
+    const int buf = it & 1, kt = tile_of(it);
+    if (it + 1 < iters) { load_tile(it + 1); cp_async_wait<1>(); } else { cp_async_wait<0>(); }
+    const int64_t slot_ahead = (tid < kKeys && it + 2 < iters) ? lookup(tile_of(it + 2)) : -1;   // in flight during this tile's math
     __syncthreads();
     const bf16* kb = Ks + buf * kKeys * QS;
     const bf16* vb = Vs + buf * kKeys * VS;
     if (few) {
       const int key0 = kt * kKeys + kq * 16;
-      if (key0 < nkeys)
+      if (key0 < nkeys && (it >= nkeep || key0 < a.keep))
         attn_tile<DMAX, VMAX, 1, VMAX / 32, QS, VS, EXT>(o, m, l, q_addr, smem_u32(kb + kq * 16 * QS + k_lane),
                                                          smem_u32(vb + kq * 16 * VS + vh * (VMAX / 2) + v_lane), key0, pos, lo, qscale, capped, cap2,
-                                                         key0 + 15 > min_pos || key0 < max_lo, tq4, bias, a.dist_rows);
+                                                         key0 + 15 > min_pos || key0 < max_lo, tq4, bias, a.dist_rows, a.keep);
     } else if (warp_has_rows) {
       // two halves of 32 keys: half the score registers of a 64-key pass (no spills under the 128-register cap)
 #pragma unroll
-      for (int hf = 0; hf < 2; ++hf)
+      for (int hf = 0; hf < 2; ++hf) {
+        if (it < nkeep && kt * kKeys + hf * 32 >= a.keep) break;   // nothing kept in this half
         attn_tile<DMAX, VMAX, 2, VMAX / 16, QS, VS, EXT>(o, m, l, q_addr, smem_u32(kb + hf * 32 * QS + k_lane), smem_u32(vb + hf * 32 * VS + v_lane),
                                                          kt * kKeys + hf * 32, pos, lo, qscale, capped, cap2,
-                                                         kt * kKeys + hf * 32 + 31 > min_pos || kt * kKeys + hf * 32 < max_lo, tq4, bias, a.dist_rows);
+                                                         kt * kKeys + hf * 32 + 31 > min_pos || kt * kKeys + hf * 32 < max_lo, tq4, bias, a.dist_rows, a.keep);
+      }
     }
-    if (tid < kKeys) slot_s[kt & 1][tid] = slot_ahead;   // tile kt's slots were consumed by load_tile(kt) an iteration ago
+    if (tid < kKeys) slot_s[buf][tid] = slot_ahead;   // this tile's slots were consumed by its load_tile an iteration ago
     __syncthreads();   // everyone is done with this buffer before the next load overwrites it
   }
 #pragma unroll
@@ -864,6 +1015,42 @@ extern "C" int nvllm_attn_rotary_store(void* q, int64_t ldq, void* k_cache, void
   return 0;
 }
 
+extern "C" int nvllm_attn_norm_rotary_store(void* q, int64_t ldq, void* k_cache, void* v_cache, int64_t k_row, int64_t v_row,
+                                            const float* proj, int64_t ldp, const float* q_norm_w, const float* k_norm_w,
+                                            float norm_eps, const int64_t* positions, const float* rope_table, int32_t rot_dims,
+                                            int32_t halves, int32_t max_pos, float* v_first, int64_t ldvf, const float* v_lambda,
+                                            const int32_t* slots, int32_t n, int32_t heads, int32_t kv_heads, int32_t dim,
+                                            int32_t vdim, int32_t dtype, void* stream) {
+  NVLLM_CHECK_ARG(n >= 0 && heads > 0 && kv_heads > 0 && dim > 0 && vdim > 0 && rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dim && max_pos > 0,
+                  NVLLM_ERR_ARG, "attn_norm_rotary_store: heads=%d/%d dim=%d vdim=%d rot_dims=%d (even, <= dim)", heads, kv_heads, dim, vdim, rot_dims);
+  NVLLM_CHECK_ARG(ldq >= static_cast<int64_t>(heads) * dim && k_row >= static_cast<int64_t>(kv_heads) * dim &&
+                      v_row >= static_cast<int64_t>(kv_heads) * vdim && (v_first == nullptr || ldvf >= static_cast<int64_t>(kv_heads) * vdim) &&
+                      ldp >= static_cast<int64_t>(heads + kv_heads) * dim + static_cast<int64_t>(kv_heads) * vdim, NVLLM_ERR_ARG,
+                  "attn_norm_rotary_store: strides");
+  NVLLM_CHECK_ARG(v_lambda == nullptr || v_first != nullptr, NVLLM_ERR_ARG, "attn_norm_rotary_store: a mixing weight without values to mix in");
+  NVLLM_CHECK_ARG(dtype == NVLLM_BF16 || dtype == NVLLM_F32, NVLLM_ERR_DTYPE, "attn_norm_rotary_store: dtype %d", dtype);
+  if (n == 0) return 0;
+  NVLLM_CHECK_ARG(q && k_cache && v_cache && proj && positions && slots && (rope_table || rot_dims == 0), NVLLM_ERR_ARG, "attn_norm_rotary_store: NULL");
+  const NormStoreArgs a{q, ldq, k_cache, v_cache, k_row, v_row, proj, ldp, q_norm_w, k_norm_w, norm_eps, positions,
+                        reinterpret_cast<const float2*>(rope_table), rot_dims, halves != 0, max_pos, v_first, ldvf, v_lambda, slots, n, heads,
+                        kv_heads, dim, vdim};
+  const int64_t items = static_cast<int64_t>(n) * (heads + 2 * kv_heads);
+  const unsigned grid = static_cast<unsigned>((items + 3) / 4);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (halves && dim % 4 == 0 && vdim % 4 == 0 && dim <= 512 && rot_dims % 8 == 0 && ldp % 4 == 0 && ldq % 4 == 0 && k_row % 4 == 0 && v_row % 4 == 0 &&
+      ldvf % 4 == 0 && aligned16(proj) && aligned16(q) && aligned16(k_cache) && aligned16(v_cache) && aligned16(rope_table) && aligned16(q_norm_w) &&
+      aligned16(k_norm_w) && aligned16(v_first)) {
+    if (dtype == NVLLM_BF16) attn_norm_rotary_store_vec_kernel<bf16><<<grid, 128, 0, st>>>(a);
+    else attn_norm_rotary_store_vec_kernel<float><<<grid, 128, 0, st>>>(a);
+    NVLLM_LAUNCH_CHECK("attn_norm_rotary_store_vec_kernel");
+    return 0;
+  }
+  if (dtype == NVLLM_BF16) attn_norm_rotary_store_kernel<bf16><<<grid, 128, 0, st>>>(a);
+  else attn_norm_rotary_store_kernel<float><<<grid, 128, 0, st>>>(a);
+  NVLLM_LAUNCH_CHECK("attn_norm_rotary_store_kernel");
+  return 0;
+}
+
 extern "C" int nvllm_capped_attention(void* out, int64_t ldo, const void* q, int64_t ldq, const float* gate, int64_t ldg,
                                       const void* k_cache, const void* v_cache, int64_t k_row, int64_t v_row,
                                       const int32_t* tok_seq, const int64_t* positions, const int32_t* block_tables,
@@ -894,7 +1081,20 @@ extern "C" int nvllm_biased_attention(void* out, int64_t ldo, const void* q, int
                                       const float* sinks, int32_t chunk, const float* head_scale, const float* dist_bias,
                                       int32_t dist_rows, const float* out_rot_table, int32_t max_pos, const int32_t* cu_tokens,
                                       int32_t n_seqs, int32_t dtype, void* stream) {
-  NVLLM_CHECK_ARG(chunk >= 0 && (dist_bias == nullptr || dist_rows > 0) && (out_rot_table == nullptr || (max_pos > 0 && vdim % 2 == 0)),
+  return nvllm_masked_attention(out, ldo, q, ldq, gate, ldg, gate_per_head, k_cache, v_cache, k_row, v_row, tok_seq, positions, block_tables,
+                                table_cap, block_size, n, heads, kv_heads, dim, vdim, scale, softcap, temp_coef, temp_every, window, 0, sinks,
+                                chunk, head_scale, dist_bias, dist_rows, out_rot_table, max_pos, cu_tokens, n_seqs, dtype, stream);
+}
+
+extern "C" int nvllm_masked_attention(void* out, int64_t ldo, const void* q, int64_t ldq, const float* gate, int64_t ldg,
+                                      int32_t gate_per_head, const void* k_cache, const void* v_cache, int64_t k_row, int64_t v_row,
+                                      const int32_t* tok_seq, const int64_t* positions, const int32_t* block_tables,
+                                      int32_t table_cap, int32_t block_size, int32_t n, int32_t heads, int32_t kv_heads, int32_t dim,
+                                      int32_t vdim, float scale, float softcap, float temp_coef, int32_t temp_every, int32_t window,
+                                      int32_t keep_first, const float* sinks, int32_t chunk, const float* head_scale,
+                                      const float* dist_bias, int32_t dist_rows, const float* out_rot_table, int32_t max_pos,
+                                      const int32_t* cu_tokens, int32_t n_seqs, int32_t dtype, void* stream) {
+  NVLLM_CHECK_ARG(chunk >= 0 && keep_first >= 0 && (dist_bias == nullptr || dist_rows > 0) && (out_rot_table == nullptr || (max_pos > 0 && vdim % 2 == 0)),
                   NVLLM_ERR_ARG, "attention: chunk=%d dist_rows=%d max_pos=%d vdim=%d (an output rotation pairs the halves of an even vdim)", chunk,
                   dist_rows, max_pos, vdim);
   NVLLM_CHECK_ARG(n >= 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && dim > 0 && vdim > 0 && vdim <= 32 * kMaxVPerLane &&
@@ -905,7 +1105,7 @@ extern "C" int nvllm_biased_attention(void* out, int64_t ldo, const void* q, int
   NVLLM_CHECK_ARG(out && q && k_cache && v_cache && tok_seq && positions && (block_tables || cu_tokens), NVLLM_ERR_ARG, "attention: NULL");
   AttnArgs a{out, ldo, q, ldq, gate, ldg, k_cache, v_cache, k_row, v_row, tok_seq, positions, block_tables, table_cap, block_size,
              n, heads, kv_heads, dim, vdim, scale, softcap, temp_coef, temp_every, window > 0 ? window : 0, sinks, gate_per_head, block_tables ? nullptr : cu_tokens,
-             chunk, head_scale, dist_bias, dist_rows, reinterpret_cast<const float2*>(out_rot_table), max_pos, 0};
+             keep_first, chunk, head_scale, dist_bias, dist_rows, reinterpret_cast<const float2*>(out_rot_table), max_pos, 0};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   // bf16 with 16-byte rows and a token range per sequence: tensor cores; everything else (f32, odd sizes): one warp per row
   const int group = heads / kv_heads;

@@ -76,7 +76,7 @@ __device__ __forceinline__ void st_smem_f32(uint32_t addr, float v) {
 template <int BN, int SK, bool SILU>
 __global__ void __launch_bounds__(256, 1)
 gemm_splitk_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_constant__ CUtensorMap tmap_w,
-                   bf16* __restrict__ y, int M, int N, int K, int64_t ldy, int num_m_tiles, int STAGES, const RowPush ps) {
+                   bf16* __restrict__ y, int M, int N, int K, int64_t ldy, int num_m_tiles, int STAGES, const RowPush ps, float glu_limit) {
   using C = SkCfg<BN>;
   extern __shared__ uint8_t smem_raw[];
   const uint32_t smem_base = (smem_u32(smem_raw) + 1023u) & ~1023u;
@@ -223,9 +223,8 @@ gemm_splitk_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_cons
         for (int e = 0; e < 8; e += 2) {  // rounding points of the unfused path: bf16 gate_up, bf16 silu(gate), bf16 product
           const uint32_t gb = pack_bf16x2(g[e], g[e + 1]);
           const uint32_t ub = pack_bf16x2(u[e], u[e + 1]);
-          const float g0 = bf16_lo(gb), g1 = bf16_hi(gb);
-          const uint32_t sb = pack_bf16x2(g0 / (1.0f + expf(-g0)), g1 / (1.0f + expf(-g1)));
-          o[e / 2] = pack_bf16x2(bf16_lo(sb) * bf16_lo(ub), bf16_hi(sb) * bf16_hi(ub));
+          const float2 p = gated_pair(gb, ub, glu_limit);
+          o[e / 2] = pack_bf16x2(p.x, p.y);
         }
         if (row < M) *reinterpret_cast<uint4*>(dst + j) = make_uint4(o[0], o[1], o[2], o[3]);
       }
@@ -303,7 +302,7 @@ int splitk_stages(int kb_per) {
 
 template <int BN, int SK, bool SILU>
 int launch_splitk(const CUtensorMap& tx, const CUtensorMap& tw, void* y, int M, int N, int K, int64_t ldy, int tiles,
-                  int num_m_tiles, cudaStream_t st, const RowPush& ps) {
+                  int num_m_tiles, cudaStream_t st, const RowPush& ps, float glu_limit = 0.f) {
   using C = SkCfg<BN>;
   auto kern = gemm_splitk_kernel<BN, SK, SILU>;
   NVLLM_SMEM_ATTR_ONCE(kern, C::smem_bytes(C::kMaxStages));
@@ -320,7 +319,7 @@ int launch_splitk(const CUtensorMap& tx, const CUtensorMap& tw, void* y, int M, 
   attr[1].val.programmaticStreamSerializationAllowed = 1;
   cfg.attrs = attr;
   cfg.numAttrs = pdl_enabled() ? 2 : 1;
-  NVLLM_CUDA(cudaLaunchKernelEx(&cfg, kern, tx, tw, static_cast<bf16*>(y), M, N, K, ldy, num_m_tiles, stages, ps));
+  NVLLM_CUDA(cudaLaunchKernelEx(&cfg, kern, tx, tw, static_cast<bf16*>(y), M, N, K, ldy, num_m_tiles, stages, ps, glu_limit));
   return 0;
 }
 
@@ -382,7 +381,7 @@ namespace nvllm {
 #endif
 
 int gemm_splitk_dispatch(void* y, const void* x, const void* w, int m, int n, int k, int64_t ldx, int64_t ldw, int64_t ldy,
-                         bool silu, int bn, int sk, cudaStream_t st, const RowPush& ps) {
+                         bool silu, int bn, int sk, cudaStream_t st, const RowPush& ps, float glu_limit) {
   CUtensorMap tx, tw;
   const int n_acc = silu ? 2 * n : n;
   if (int rc = make_tmap_bf16_2d(&tx, x, m, k, ldx, 128)) return rc;
@@ -390,7 +389,7 @@ int gemm_splitk_dispatch(void* y, const void* x, const void* w, int m, int n, in
   const int mt = (m + 127) / 128, tiles = mt * (n_acc / bn);
 #define NVLLM_SK(BNV, SKV)                                                                                   \
   if (bn == BNV && sk == SKV)                                                                                \
-    return silu ? launch_splitk<BNV, SKV, true>(tx, tw, y, m, n, k, ldy, tiles, mt, st, RowPush{})                      \
+    return silu ? launch_splitk<BNV, SKV, true>(tx, tw, y, m, n, k, ldy, tiles, mt, st, RowPush{}, glu_limit)                      \
                 : launch_splitk<BNV, SKV, false>(tx, tw, y, m, n, k, ldy, tiles, mt, st, ps)
   NVLLM_SK(256, 8); NVLLM_SK(256, 4); NVLLM_SK(256, 2);
   NVLLM_SK(128, 8); NVLLM_SK(128, 4); NVLLM_SK(128, 2);

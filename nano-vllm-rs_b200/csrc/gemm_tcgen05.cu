@@ -74,7 +74,7 @@ __device__ __forceinline__ void store_row32<float>(float* dst, const uint32_t (&
 }
 
 // SILU == true: w = [gate (N rows) | up (N rows)]; the B tile is staged as BN/2 gate rows + the matching BN/2 up rows and
-// the epilogue writes y[:, n_tile*BN/2 + c] = silu(gate) * up (see gemm_tcgen05_2cta.cu for the CTA-pair variant).
+// the epilogue writes y[:, n_tile*BN/2 + c] = silu(gate) * up, or with glu_limit > 0 the clamped gate of gated_pair (see gemm_tcgen05_2cta.cu for the CTA-pair variant).
 // Optional qkv epilogue (ROPE mode, BN == 128 == head_dim): each output tile is one head of the packed [q | k | v] row,
 // and each epilogue thread owns that head for one token.  It applies what Qwen3Attention::forward does between qkv_proj
 // and Attention::forward (qwen3.rs:219-229) plus Attention::store_kv_cache (attention.rs:150-174): round to bf16 (the
@@ -101,7 +101,7 @@ __global__ void __launch_bounds__(256, 1)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_constant__ CUtensorMap tmap_w,
                     OutT* __restrict__ y, int M, int N, int K, int64_t ldy, int num_m_tiles, int num_tiles,
                     const RopeEpi re = RopeEpi{}, int STAGES = GemmCfg<BN>::kStages, const RowPush ps = RowPush{},
-                    const int32_t* __restrict__ tile_group = nullptr, int group_rows = 0) {
+                    const int32_t* __restrict__ tile_group = nullptr, int group_rows = 0, float glu_limit = 0.f) {
   // tile_group != nullptr (expert layers): 128-row tile m uses the weight block of group tile_group[m], i.e. rows
   // [group * group_rows, ...) of w; an unused tile (group < 0) runs against group 0 and its rows are never read.
   using C = GemmCfg<BN>;  // STAGES <= C::kStages: ring depth of this launch (fewer stages -> two CTAs per SM, see launch_gemm)
@@ -309,10 +309,9 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_con
           for (int e = 0; e < 32; e += 2) {  // rounding points of the unfused path: bf16 gate_up, bf16 silu(gate)
             const uint32_t gb = pack_bf16x2(__uint_as_float(g[e]), __uint_as_float(g[e + 1]));
             const uint32_t ub = pack_bf16x2(__uint_as_float(u[e]), __uint_as_float(u[e + 1]));
-            const float g0 = bf16_lo(gb), g1 = bf16_hi(gb);
-            const uint32_t sb = pack_bf16x2(g0 / (1.0f + expf(-g0)), g1 / (1.0f + expf(-g1)));
-            g[e] = __float_as_uint(bf16_lo(sb) * bf16_lo(ub));
-            g[e + 1] = __float_as_uint(bf16_hi(sb) * bf16_hi(ub));
+            const float2 p = gated_pair(gb, ub, glu_limit);
+            g[e] = __float_as_uint(p.x);
+            g[e + 1] = __float_as_uint(p.y);
           }
           const int col0 = n_tile * (BN / 2) + c * 32;
           if (row < M && col0 < N) store_row32<OutT>(y + row * ldy + col0, g, col0, N);
@@ -351,7 +350,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_con
 template <int BN, typename OutT, bool SILU = false, int CN = 1, bool ROPE = false>
 static int launch_gemm(const CUtensorMap& tx, const CUtensorMap& tw, void* y, int M, int N, int K, int64_t ldy,
                        cudaStream_t st, const RopeEpi& re = RopeEpi{}, const RowPush& ps = RowPush{},
-                       const int32_t* tile_group = nullptr, int group_rows = 0) {
+                       const int32_t* tile_group = nullptr, int group_rows = 0, float glu_limit = 0.f) {
   using C = GemmCfg<BN>;
   auto kern = gemm_tcgen05_kernel<BN, OutT, SILU, CN, ROPE>;
   NVLLM_SMEM_ATTR_ONCE(kern, C::kSmemBytes);
@@ -371,7 +370,7 @@ static int launch_gemm(const CUtensorMap& tx, const CUtensorMap& tw, void* y, in
   const int smem = C::kSmemBytes - (C::kStages - stages) * C::kStageBytes;
   if constexpr (CN == 1) {
     NVLLM_CUDA(launch_pdl(kern, dim3(clusters), dim3(256), smem, st, tx, tw, static_cast<OutT*>(y), M, N, K, ldy,
-                          num_m_tiles, num_tiles, re, stages, ps, tile_group, group_rows));
+                          num_m_tiles, num_tiles, re, stages, ps, tile_group, group_rows, glu_limit));
   } else {
     cudaLaunchConfig_t cfg{};
     cfg.gridDim = dim3(clusters * CN);
@@ -386,7 +385,7 @@ static int launch_gemm(const CUtensorMap& tx, const CUtensorMap& tw, void* y, in
     cfg.attrs = attr;
     cfg.numAttrs = pdl_enabled() ? 2 : 1;
     NVLLM_CUDA(cudaLaunchKernelEx(&cfg, kern, tx, tw, static_cast<OutT*>(y), M, N, K, ldy, num_m_tiles, num_tiles, re,
-                                  static_cast<int>(C::kStages), ps, tile_group, group_rows));
+                                  static_cast<int>(C::kStages), ps, tile_group, group_rows, glu_limit));
   }
   return 0;
 }
@@ -423,12 +422,12 @@ int gemm_2cta_dispatch(void* y, const void* x, const void* w, int m, int n, int 
                        int64_t ldy, int out_dtype, cudaStream_t st);  // gemm_tcgen05_2cta.cu
 
 int gemm_silu_2cta_dispatch(void* y, const void* x, const void* w, int m, int inter, int k, int64_t ldx, int64_t ldw,
-                            int64_t ldy, cudaStream_t st);  // gemm_tcgen05_2cta.cu
+                            int64_t ldy, float glu_limit, cudaStream_t st);  // gemm_tcgen05_2cta.cu
 
 // gemm_splitk.cu: cluster split-K for decode-sized projections (m <= 256)
 bool splitk_choose(int m, int n_acc, int k, bool silu, int bn_default, int* out_bn, int* out_sk);
 int gemm_splitk_dispatch(void* y, const void* x, const void* w, int m, int n, int k, int64_t ldx, int64_t ldw, int64_t ldy,
-                         bool silu, int bn, int sk, cudaStream_t st, const RowPush& ps = RowPush{});
+                         bool silu, int bn, int sk, cudaStream_t st, const RowPush& ps = RowPush{}, float glu_limit = 0.f);
 
 static bool use_2cta();
 // CTA pairs pay off once there are at least two 256-row tiles or the problem is large enough to fill the machine with
@@ -540,10 +539,37 @@ extern "C" int nvllm_gemm_bf16_grouped(void* y, const void* x, const void* w, in
   }
 }
 
+// The grouped GEMM over [gate (inter rows) | up (inter rows)] blocks with the gate in the epilogue: y [max_rows, inter].
+extern "C" int nvllm_gemm_glu_bf16_grouped(void* y, const void* x, const void* w, int32_t max_rows, int32_t inter, int32_t k,
+                                           int32_t groups, int64_t ldx, int64_t ldw, int64_t ldy, const int32_t* tile_group,
+                                           float limit, void* stream) {
+  using namespace nvllm;
+  NVLLM_CHECK_ARG(max_rows >= 0 && max_rows % 128 == 0 && inter > 0 && k > 0 && groups > 0 && k % 64 == 0 && inter % 64 == 0, NVLLM_ERR_ARG,
+                  "gemm_glu_grouped: max_rows=%d (multiple of 128) inter=%d (%% 64) k=%d (%% 64) groups=%d", max_rows, inter, k, groups);
+  NVLLM_CHECK_ARG(ldx >= k && ldw >= k && ldy >= inter && ldx % 8 == 0 && ldw % 8 == 0 && ldy % 8 == 0, NVLLM_ERR_ALIGN,
+                  "gemm_glu_grouped: leading dimensions");
+  if (max_rows == 0) return 0;
+  NVLLM_CHECK_ARG(y && x && w && tile_group && aligned16(y) && aligned16(x) && aligned16(w), NVLLM_ERR_ALIGN, "gemm_glu_grouped: pointers");
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const int bn = inter >= 128 ? 256 : 128;
+  CUtensorMap tx, tw;
+  if (int rc = make_tmap_bf16_2d(&tx, x, max_rows, k, ldx, 128)) return rc;
+  if (int rc = make_tmap_bf16_2d(&tw, w, static_cast<int64_t>(groups) * 2 * inter, k, ldw, bn / 2)) return rc;
+  if (bn == 256) return launch_gemm<256, bf16, true>(tx, tw, y, max_rows, inter, k, ldy, st, RopeEpi{}, RowPush{}, tile_group, 2 * inter, limit);
+  return launch_gemm<128, bf16, true>(tx, tw, y, max_rows, inter, k, ldy, st, RopeEpi{}, RowPush{}, tile_group, 2 * inter, limit);
+}
+
 // MergedColumnParallelLinear::forward + SiluAndMul::forward in one call (linear.rs:437-439 + activation.rs:46-63).
 extern "C" int nvllm_gemm_silu_mul_bf16(void* out, const void* x, const void* w_gate_up, int32_t m, int32_t inter,
                                         int32_t k, int64_t ldx, int64_t ldw, int64_t ldout, void* workspace,
                                         size_t workspace_bytes, void* stream) {
+  return nvllm_gemm_glu_bf16(out, x, w_gate_up, m, inter, k, ldx, ldw, ldout, 0.f, workspace, workspace_bytes, stream);
+}
+
+// The same with the gate as a parameter: limit <= 0 SiLU, limit > 0 the clamped gate (gated_pair, common.cuh).
+extern "C" int nvllm_gemm_glu_bf16(void* out, const void* x, const void* w_gate_up, int32_t m, int32_t inter, int32_t k,
+                                   int64_t ldx, int64_t ldw, int64_t ldout, float limit, void* workspace,
+                                   size_t workspace_bytes, void* stream) {
   using namespace nvllm;
   NVLLM_CHECK_ARG(m >= 0 && inter > 0 && k > 0 && k % 64 == 0 && inter % 8 == 0, NVLLM_ERR_ARG,
                   "gemm_silu_mul: m=%d inter=%d k=%d (k %% 64, inter %% 8)", m, inter, k);
@@ -559,17 +585,17 @@ extern "C" int nvllm_gemm_silu_mul_bf16(void* out, const void* x, const void* w_
     {
       int sbn = 0, ssk = 0;
       if (splitk_choose(m, 2 * inter, k, true, bn, &sbn, &ssk))
-        return gemm_splitk_dispatch(out, x, w_gate_up, m, inter, k, ldx, ldw, ldout, true, sbn, ssk, st);
+        return gemm_splitk_dispatch(out, x, w_gate_up, m, inter, k, ldx, ldw, ldout, true, sbn, ssk, st, RowPush{}, limit);
     }
-    if (want_2cta(m, 2 * inter, k)) return gemm_silu_2cta_dispatch(out, x, w_gate_up, m, inter, k, ldx, ldw, ldout, st);
+    if (want_2cta(m, 2 * inter, k)) return gemm_silu_2cta_dispatch(out, x, w_gate_up, m, inter, k, ldx, ldw, ldout, limit, st);
     CUtensorMap tx, tw;
     if (int rc = make_tmap_bf16_2d(&tx, x, m, k, ldx, 128)) return rc;
     if (int rc = make_tmap_bf16_2d(&tw, w_gate_up, 2 * static_cast<int64_t>(inter), k, ldw, bn / 2)) return rc;
     switch (bn) {
-      case 256: return launch_gemm<256, bf16, true>(tx, tw, out, m, inter, k, ldout, st);
-      case 192: return launch_gemm<192, bf16, true>(tx, tw, out, m, inter, k, ldout, st);
-      case 128: return launch_gemm<128, bf16, true>(tx, tw, out, m, inter, k, ldout, st);
-      default: return launch_gemm<64, bf16, true>(tx, tw, out, m, inter, k, ldout, st);
+      case 256: return launch_gemm<256, bf16, true>(tx, tw, out, m, inter, k, ldout, st, RopeEpi{}, RowPush{}, nullptr, 0, limit);
+      case 192: return launch_gemm<192, bf16, true>(tx, tw, out, m, inter, k, ldout, st, RopeEpi{}, RowPush{}, nullptr, 0, limit);
+      case 128: return launch_gemm<128, bf16, true>(tx, tw, out, m, inter, k, ldout, st, RopeEpi{}, RowPush{}, nullptr, 0, limit);
+      default: return launch_gemm<64, bf16, true>(tx, tw, out, m, inter, k, ldout, st, RopeEpi{}, RowPush{}, nullptr, 0, limit);
     }
   }
   // odd intermediate sizes: plain GEMM into the workspace, then the SiLU*mul kernel
@@ -578,6 +604,7 @@ extern "C" int nvllm_gemm_silu_mul_bf16(void* out, const void* x, const void* w_
                   "gemm_silu_mul: workspace %zu < %zu bytes", workspace_bytes, need);
   NVLLM_CHECK_ARG(ldout == inter, NVLLM_ERR_ARG, "gemm_silu_mul: unfused path needs a contiguous output");
   if (int rc = nvllm_gemm_bf16(workspace, x, w_gate_up, m, 2 * inter, k, ldx, ldw, 2 * inter, NVLLM_BF16, nullptr, 0, stream)) return rc;
+  if (limit > 0.f) return nvllm_glu_clamped(out, workspace, m, inter, limit, NVLLM_BF16, stream);
   return nvllm_silu_mul(out, workspace, m, inter, NVLLM_BF16, stream);
 }
 

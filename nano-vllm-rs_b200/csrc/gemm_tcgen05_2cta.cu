@@ -49,11 +49,11 @@ __device__ __forceinline__ void store_row32_2(OutT* dst, const uint32_t (&r)[32]
 // SILU == true: w is the packed [gate (N rows) | up (N rows)] matrix of MergedColumnParallelLinear (linear.rs:421-433);
 // the leader CTA stages BN/2 gate rows, its peer the matching BN/2 up rows, so accumulator columns [0, BN/2) are gate and
 // [BN/2, BN) are up for the same BN/2 output features, and the epilogue writes y[:, n_tile*BN/2 + c] = silu(gate)*up
-// (SiluAndMul::forward, activation.rs:46-63) without the [M, 2N] intermediate ever reaching HBM.  N = output features.
+// (SiluAndMul::forward, activation.rs:46-63; glu_limit > 0: the clamped gate of gated_pair) without the [M, 2N] intermediate ever reaching HBM.  N = output features.
 template <int BN, typename OutT, bool SILU>
 __global__ void __launch_bounds__(256, 1)
 gemm_tcgen05_2cta_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_constant__ CUtensorMap tmap_w,
-                         OutT* __restrict__ y, int M, int N, int K, int64_t ldy, int num_m_tiles, int num_tiles) {
+                         OutT* __restrict__ y, int M, int N, int K, int64_t ldy, int num_m_tiles, int num_tiles, float glu_limit) {
   using C = Gemm2Cfg<BN>;
   constexpr int STAGES = C::kStages;
   extern __shared__ uint8_t smem_raw[];
@@ -162,10 +162,9 @@ gemm_tcgen05_2cta_kernel(const __grid_constant__ CUtensorMap tmap_x, const __gri
             // same rounding points as the unfused path: gate_up is a bf16 tensor, silu(gate) is a bf16 tensor
             const uint32_t gb = pack_bf16x2(__uint_as_float(g[e]), __uint_as_float(g[e + 1]));
             const uint32_t ub = pack_bf16x2(__uint_as_float(u[e]), __uint_as_float(u[e + 1]));
-            const float g0 = bf16_lo(gb), g1 = bf16_hi(gb);
-            const uint32_t sb = pack_bf16x2(g0 / (1.0f + expf(-g0)), g1 / (1.0f + expf(-g1)));
-            g[e] = __float_as_uint(bf16_lo(sb) * bf16_lo(ub));
-            g[e + 1] = __float_as_uint(bf16_hi(sb) * bf16_hi(ub));
+            const float2 p = gated_pair(gb, ub, glu_limit);
+            g[e] = __float_as_uint(p.x);
+            g[e + 1] = __float_as_uint(p.y);
           }
           const int col0 = n_tile * (BN / 2) + c * 32;
           if (row < M && col0 < N) store_row32_2<OutT>(y + row * ldy + col0, g, col0, N);
@@ -196,7 +195,7 @@ gemm_tcgen05_2cta_kernel(const __grid_constant__ CUtensorMap tmap_x, const __gri
 
 template <int BN, typename OutT, bool SILU = false>
 static int launch_gemm2(const CUtensorMap& tx, const CUtensorMap& tw, void* y, int M, int N, int K, int64_t ldy,
-                        cudaStream_t st) {
+                        cudaStream_t st, float glu_limit = 0.f) {
   using C = Gemm2Cfg<BN>;
   auto kern = gemm_tcgen05_2cta_kernel<BN, OutT, SILU>;
   NVLLM_SMEM_ATTR_ONCE(kern, C::kSmemBytes);
@@ -217,7 +216,7 @@ static int launch_gemm2(const CUtensorMap& tx, const CUtensorMap& tw, void* y, i
   attr[1].val.programmaticStreamSerializationAllowed = 1;
   cfg.attrs = attr;
   cfg.numAttrs = pdl_enabled() ? 2 : 1;
-  NVLLM_CUDA(cudaLaunchKernelEx(&cfg, kern, tx, tw, static_cast<OutT*>(y), M, N, K, ldy, num_m_tiles, num_tiles));
+  NVLLM_CUDA(cudaLaunchKernelEx(&cfg, kern, tx, tw, static_cast<OutT*>(y), M, N, K, ldy, num_m_tiles, num_tiles, glu_limit));
   return 0;
 }
 
@@ -262,9 +261,9 @@ int gemm_2cta_dispatch(void* y, const void* x, const void* w, int m, int n, int 
 #undef NVLLM_G2
 }
 
-// y[M, inter] = silu(x . Wgate^T) * (x . Wup^T) with w = [Wgate | Wup] packed row-wise ([2*inter, K]).
+// y[M, inter] = silu(x . Wgate^T) * (x . Wup^T) (or the clamped gate) with w = [Wgate | Wup] packed row-wise ([2*inter, K]).
 int gemm_silu_2cta_dispatch(void* y, const void* x, const void* w, int m, int inter, int k, int64_t ldx, int64_t ldw,
-                            int64_t ldy, cudaStream_t st) {
+                            int64_t ldy, float glu_limit, cudaStream_t st) {
   // accumulator tile BN covers BN/2 output features; reuse the tile heuristic on the 2*inter accumulator columns
   const int bn = pick_bn_2cta(m, 2 * inter);
   NVLLM_CHECK_ARG(inter % (bn / 2) == 0 || true, NVLLM_ERR_ARG, "gemm_silu: inter");
@@ -272,9 +271,9 @@ int gemm_silu_2cta_dispatch(void* y, const void* x, const void* w, int m, int in
   if (int rc = make_tmap_bf16_2d(&tx, x, m, k, ldx, 128)) return rc;
   if (int rc = make_tmap_bf16_2d(&tw, w, 2 * static_cast<int64_t>(inter), k, ldw, bn / 2)) return rc;
   switch (bn) {
-    case 256: return launch_gemm2<256, bf16, true>(tx, tw, y, m, inter, k, ldy, st);
-    case 128: return launch_gemm2<128, bf16, true>(tx, tw, y, m, inter, k, ldy, st);
-    default: return launch_gemm2<64, bf16, true>(tx, tw, y, m, inter, k, ldy, st);
+    case 256: return launch_gemm2<256, bf16, true>(tx, tw, y, m, inter, k, ldy, st, glu_limit);
+    case 128: return launch_gemm2<128, bf16, true>(tx, tw, y, m, inter, k, ldy, st, glu_limit);
+    default: return launch_gemm2<64, bf16, true>(tx, tw, y, m, inter, k, ldy, st, glu_limit);
   }
 }
 

@@ -27,14 +27,29 @@ template <typename T> __device__ __forceinline__ void stf(T* p, float v);
 template <> __device__ __forceinline__ void stf<float>(float* p, float v) { *p = v; }
 template <> __device__ __forceinline__ void stf<bf16>(bf16* p, float v) { *p = __float2bfloat16_rn(v); }
 
-// table[p][i] = (cos, sin)(p * base^(-2i/dims)), i < dims/2, angles in f64
-__global__ void rope_table_interleaved_kernel(float2* __restrict__ tab, int max_pos, int half, int dims, double base) {
+// Wavelength-dependent scaling of the rotary frequencies; off while factor <= 0.  A wave that turns more than `high` times
+// within `original` positions keeps its frequency, one that turns fewer than `low` times is slowed down `factor` times,
+// between them the two are blended linearly in the number of turns.
+struct RopeScaling { double factor, low, high, original; };
+
+// table[p][i] = (cos, sin)(p * f_i), f_i = base^(-2i/dims) (scaled), i < dims/2, angles in f64
+__global__ void rope_table_interleaved_kernel(float2* __restrict__ tab, int max_pos, int half, int dims, double base, const RopeScaling sc) {
   const int64_t total = static_cast<int64_t>(max_pos) * half;
   for (int64_t e = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; e < total;
        e += static_cast<int64_t>(gridDim.x) * blockDim.x) {
     const int64_t p = e / half;
     const int i = static_cast<int>(e - p * half);
-    const double f = pow(base, -2.0 * i / dims), a = static_cast<double>(p) * f;
+    double f = pow(base, -2.0 * i / dims);
+    if (sc.factor > 0.0) {
+      const double wave = 6.283185307179586476925 / f;
+      if (wave > sc.original / sc.low) {
+        f /= sc.factor;
+      } else if (wave >= sc.original / sc.high) {
+        const double s = sc.high > sc.low ? (sc.original / wave - sc.low) / (sc.high - sc.low) : 1.0;
+        f = (1.0 - s) * f / sc.factor + s * f;
+      }
+    }
+    const double a = static_cast<double>(p) * f;
     tab[e] = make_float2(static_cast<float>(cos(a)), static_cast<float>(sin(a)));
   }
 }
@@ -564,13 +579,20 @@ int dispatch_attn(const AttnArgs& a, cudaStream_t st) {
 using namespace nvllm;
 
 extern "C" int nvllm_rope_table_interleaved(float* cos_sin, int32_t max_pos, int32_t dims, double base, void* stream) {
+  return nvllm_rope_table_scaled(cos_sin, max_pos, dims, base, 0.0, 1.0, 2.0, 1.0, stream);
+}
+
+extern "C" int nvllm_rope_table_scaled(float* cos_sin, int32_t max_pos, int32_t dims, double base, double factor, double low, double high,
+                                       double original, void* stream) {
+  NVLLM_CHECK_ARG(factor <= 0.0 || (low > 0.0 && high >= low && original > 0.0), NVLLM_ERR_ARG,
+                  "rope_table_scaled: factor=%g low=%g high=%g original=%g", factor, low, high, original);
   NVLLM_CHECK_ARG(cos_sin && max_pos > 0 && dims > 0 && dims % 2 == 0 && base > 0, NVLLM_ERR_ARG,
                   "rope_table_interleaved: max_pos=%d dims=%d (even) base=%g", max_pos, dims, base);
   const int64_t total = static_cast<int64_t>(max_pos) * (dims / 2);
   int64_t blocks = (total + 255) / 256;
   if (blocks > sm_count() * 16) blocks = sm_count() * 16;
   rope_table_interleaved_kernel<<<static_cast<unsigned>(blocks), 256, 0, static_cast<cudaStream_t>(stream)>>>(
-      reinterpret_cast<float2*>(cos_sin), max_pos, dims / 2, dims, base);
+      reinterpret_cast<float2*>(cos_sin), max_pos, dims / 2, dims, base, RopeScaling{factor, low, high, original});
   NVLLM_LAUNCH_CHECK("rope_table_interleaved_kernel");
   return 0;
 }

@@ -30,14 +30,6 @@ template <> __device__ __forceinline__ void stf<bf16>(bf16* p, float v) { *p = _
 
 constexpr int BM = 32, BN = 64, BK = 32;
 
-// GLU epilogue of the gated feed-forward used by the mixture-of-experts layers:
-//   g = min(gate, limit), u = clamp(up, -limit, limit), out = g * sigmoid(1.702 g) * (u + 1)
-__device__ __forceinline__ float glu_clamped(float g, float u, float limit) {
-  g = fminf(g, limit);
-  u = fminf(fmaxf(u, -limit), limit);
-  return g * (1.0f / (1.0f + expf(-1.702f * g))) * (u + 1.0f);
-}
-
 template <typename TI, typename TO, bool GLU>
 __global__ void __launch_bounds__(256) linear_tile_kernel(const LinArgs a) {
   __shared__ float xs[BM][BK + 1];

@@ -7,7 +7,9 @@
 //   nvllm_linear_recurrence   S_t = a_t S_(t-1) + b_t k_t v_t^T,   y_t = S_t^T q_t + d v_t        (S: [dk, dv] per head)
 //       covers state-space duality (k = B, q = C, v = x, a = exp(-exp(A_log) dt), b = dt, d = D; B and C shared by the heads
 //       of a group) and retention (a = a constant per head, b = 1, d = 0)
-//   nvllm_gated_delta_recurrence   the gated delta rule with a decay per key channel:  S <- diag(g_t) S,
+//   nvllm_channel_recurrence  the same with a decay per key channel (gated linear attention), S_t = diag(a_t) S_(t-1) + k_t v_t^T;
+//       nvllm_low_rank_decay makes its decays, sigmoid(A2 a1 + b)^(1/tau)
+//   nvllm_gated_delta_recurrence   the gated delta rule with a decay per key channel (nvllm_head_delta_recurrence: per head):  S <- diag(g_t) S,
 //       u = beta_t (v_t - S^T k_t),  S <- S + k_t u^T,  y_t = S^T q_t;  nvllm_delta_prepare makes its inputs (unit-length q and k,
 //       beta = sigmoid, g = exp(-exp(A_log) softplus(. + dt_bias)))
 //   nvllm_causal_conv         per-channel convolution over the last `taps` tokens (+ bias, SiLU); the slot keeps the window's
@@ -28,12 +30,13 @@ struct RecArgs {
   float* y; int64_t ldy;
   const float *q, *k, *v; int64_t ldq, ldk, ldv;
   int group_div;                 // head h reads q / k of group h / group_div
-  const float* decay; int decay_ld;   // [n, heads] (decay_ld = heads) or [heads] (decay_ld = 0)
+  const float* decay; int64_t decay_ld;   // [n, heads] (decay_ld = heads) or [heads] (decay_ld = 0); per channel: [n, heads * dk], rows decay_ld apart
   const float* step; int step_ld;     // same, or null (1)
   const float* skip;                  // [heads] or null (0)
   float* state;                       // [slots, heads, dk, dv]
   const int32_t *seq_slot, *cu_tokens; const int64_t* positions;
   int heads, dk, dv;
+  float q_scale;                      // factor on the read-out (a constant scale of the queries)
 };
 
 constexpr int kRecTile = 16;  // tokens per stage
@@ -47,14 +50,15 @@ __device__ __forceinline__ void cp_async_4(uint32_t smem_addr, const void* gptr)
 // kRecTile tokens' k, q (rows of dk), v, a, b are staged in shared memory with cp.async, two stages deep: the copies of the
 // next stage fly while the current stage's tokens are stepped through, and the steps themselves need no synchronisation.  NSL row
 // slices of one column sit in neighbouring lanes and are summed with shuffles.  vec: rows are 16-byte multiples.
-template <int NPT, int NSL, int PP>
+// CHD: one decay per key channel (a row of dk values per token and head, staged beside k and q) instead of one per head.
+template <int NPT, int NSL, int PP, bool CHD>
 __global__ void __launch_bounds__(512) linear_recurrence_kernel(const RecArgs a, int pb, int vec) {
   extern __shared__ __align__(16) float sm[];
   // a row of k (or q) in shared memory: NSL slices of NPT values, each followed by 4 floats of padding, so that the NSL
   // 16-byte broadcast reads of one warp instruction (one per slice) fall into different banks
   constexpr int SL = NPT + 4, DKP = SL * NSL;
   const int pbp = (pb + 3) & ~3;
-  const int stage = kRecTile * (2 * DKP + pbp + 2);
+  const int stage = kRecTile * ((CHD ? 3 : 2) * DKP + pbp + 2);
   const int h = blockIdx.x, s = blockIdx.y, p0 = blockIdx.z * pb;
   // the thread's PP columns lie pb / PP apart, so that neighbouring threads hold neighbouring columns (coalesced state)
   const int tid = threadIdx.x, ns = tid % NSL, pl = tid / NSL, p = p0 + pl, half = (pb + PP - 1) / PP;
@@ -75,12 +79,13 @@ __global__ void __launch_bounds__(512) linear_recurrence_kernel(const RecArgs a,
   // both stages start as zeros (rows beyond dk and columns beyond dv stay zero) with a step of 1
   for (int e = tid; e < 2 * stage; e += blockDim.x) sm[e] = 0.f;
   __syncthreads();
-  if (a.step == nullptr && tid < 2 * kRecTile) sm[(tid / kRecTile) * stage + kRecTile * (2 * DKP + pbp) + kRecTile + tid % kRecTile] = 1.f;
+  if (a.step == nullptr && tid < 2 * kRecTile) sm[(tid / kRecTile) * stage + kRecTile * ((CHD ? 3 : 2) * DKP + pbp) + kRecTile + tid % kRecTile] = 1.f;
   const int ncol = min(pb, a.dv - p0);
   auto issue = [&](int tb, int buf) {
     float* ks = sm + buf * stage;
     float* qs = ks + kRecTile * DKP;
-    float* vs = qs + kRecTile * DKP;
+    float* gs = qs + kRecTile * DKP;               // CHD only
+    float* vs = gs + (CHD ? kRecTile * DKP : 0);
     float* as = vs + kRecTile * pbp;
     float* bs = as + kRecTile;
     const int cnt = min(kRecTile, t1 - tb);
@@ -92,6 +97,7 @@ __global__ void __launch_bounds__(512) linear_recurrence_kernel(const RecArgs a,
         const int dst = tt * DKP + (c * 4 / NPT) * SL + (c * 4) % NPT;
         cp_async_16(smem_u32(ks + dst), a.k + t * a.ldk + static_cast<int64_t>(g) * a.dk + c * 4, 16);
         cp_async_16(smem_u32(qs + dst), a.q + t * a.ldq + static_cast<int64_t>(g) * a.dk + c * 4, 16);
+        if (CHD) cp_async_16(smem_u32(gs + dst), a.decay + t * a.decay_ld + static_cast<int64_t>(h) * a.dk + c * 4, 16);
       }
       for (int e = tid; e < cnt * vch; e += blockDim.x) {
         const int tt = e / vch, c = e - tt * vch;
@@ -104,6 +110,7 @@ __global__ void __launch_bounds__(512) linear_recurrence_kernel(const RecArgs a,
         const int dst = tt * DKP + (n / NPT) * SL + n % NPT;
         cp_async_4(smem_u32(ks + dst), a.k + t * a.ldk + static_cast<int64_t>(g) * a.dk + n);
         cp_async_4(smem_u32(qs + dst), a.q + t * a.ldq + static_cast<int64_t>(g) * a.dk + n);
+        if (CHD) cp_async_4(smem_u32(gs + dst), a.decay + t * a.decay_ld + static_cast<int64_t>(h) * a.dk + n);
       }
       for (int e = tid; e < cnt * ncol; e += blockDim.x) {
         const int tt = e / ncol, c = e - tt * ncol;
@@ -112,7 +119,7 @@ __global__ void __launch_bounds__(512) linear_recurrence_kernel(const RecArgs a,
     }
     if (tid < cnt) {
       const int64_t t = tb + tid;
-      cp_async_4(smem_u32(as + tid), a.decay + (a.decay_ld ? t * a.decay_ld + h : h));
+      if (!CHD) cp_async_4(smem_u32(as + tid), a.decay + (a.decay_ld ? t * a.decay_ld + h : h));
       if (a.step) cp_async_4(smem_u32(bs + tid), a.step + (a.step_ld ? t * a.step_ld + h : h));
     }
     cp_async_commit();
@@ -136,32 +143,34 @@ __global__ void __launch_bounds__(512) linear_recurrence_kernel(const RecArgs a,
     __syncthreads();
     const float* ks = sm + buf * stage;
     const float* qs = ks + kRecTile * DKP;
-    const float* vs = qs + kRecTile * DKP;
+    const float* gs = qs + kRecTile * DKP;
+    const float* vs = gs + (CHD ? kRecTile * DKP : 0);
     const float* as = vs + kRecTile * pbp;
     const float* bs = as + kRecTile;
     for (int tt = 0; tt < cnt; ++tt) {
-      const float av = as[tt], bt = bs[tt];
+      const float av = CHD ? 0.f : as[tt], bt = bs[tt];
       float xv[PP], bv[PP], acc[PP];
 #pragma unroll
       for (int j = 0; j < PP; ++j) { xv[j] = vs[tt * pbp + (live[j] ? pl + j * half : 0)]; bv[j] = bt * xv[j]; acc[j] = 0.f; }
       const float4* kr = reinterpret_cast<const float4*>(ks + tt * DKP + ns * SL);   // broadcast reads, 16 bytes each
       const float4* qr = reinterpret_cast<const float4*>(qs + tt * DKP + ns * SL);
+      const float4* gr = reinterpret_cast<const float4*>(gs + tt * DKP + ns * SL);
 #pragma unroll
       for (int i = 0; i < NPT / 4; ++i) {
-        const float4 k4 = kr[i], q4 = qr[i];
+        const float4 k4 = kr[i], q4 = qr[i], g4 = CHD ? gr[i] : make_float4(av, av, av, av);
 #pragma unroll
         for (int j = 0; j < PP; ++j) {
-          S[j][4 * i] = fmaf(av, S[j][4 * i], bv[j] * k4.x);         acc[j] = fmaf(S[j][4 * i], q4.x, acc[j]);
-          S[j][4 * i + 1] = fmaf(av, S[j][4 * i + 1], bv[j] * k4.y); acc[j] = fmaf(S[j][4 * i + 1], q4.y, acc[j]);
-          S[j][4 * i + 2] = fmaf(av, S[j][4 * i + 2], bv[j] * k4.z); acc[j] = fmaf(S[j][4 * i + 2], q4.z, acc[j]);
-          S[j][4 * i + 3] = fmaf(av, S[j][4 * i + 3], bv[j] * k4.w); acc[j] = fmaf(S[j][4 * i + 3], q4.w, acc[j]);
+          S[j][4 * i] = fmaf(g4.x, S[j][4 * i], bv[j] * k4.x);         acc[j] = fmaf(S[j][4 * i], q4.x, acc[j]);
+          S[j][4 * i + 1] = fmaf(g4.y, S[j][4 * i + 1], bv[j] * k4.y); acc[j] = fmaf(S[j][4 * i + 1], q4.y, acc[j]);
+          S[j][4 * i + 2] = fmaf(g4.z, S[j][4 * i + 2], bv[j] * k4.z); acc[j] = fmaf(S[j][4 * i + 2], q4.z, acc[j]);
+          S[j][4 * i + 3] = fmaf(g4.w, S[j][4 * i + 3], bv[j] * k4.w); acc[j] = fmaf(S[j][4 * i + 3], q4.w, acc[j]);
         }
       }
 #pragma unroll
       for (int j = 0; j < PP; ++j) {
 #pragma unroll
         for (int o = 1; o < NSL; o <<= 1) acc[j] += __shfl_xor_sync(0xffffffffu, acc[j], o);
-        if (live[j] && ns == 0) a.y[(tb + tt) * a.ldy + static_cast<int64_t>(h) * a.dv + p + j * half] = fmaf(d, xv[j], acc[j]);
+        if (live[j] && ns == 0) a.y[(tb + tt) * a.ldy + static_cast<int64_t>(h) * a.dv + p + j * half] = fmaf(d, xv[j], acc[j] * a.q_scale);
       }
     }
     __syncthreads();   // the copy issued in the next iteration overwrites this stage
@@ -180,7 +189,7 @@ struct DeltaArgs {
   float* y; int64_t ldy;
   const float *q, *k, *v; int64_t ldq, ldk, ldv;
   int group_div;                       // head h reads q / k of group h / group_div
-  const float* decay; int64_t ldd;     // [n, heads * dk]: decay of every key channel
+  const float* decay; int64_t ldd;     // [n, heads * dk]: decay of every key channel; HEADG: [n, heads]
   const float* beta; int64_t ldb;      // [n, heads]
   float* state;                        // [slots, heads, dk, dv]
   const int32_t *seq_slot, *cu_tokens; const int64_t* positions;
@@ -191,13 +200,13 @@ struct DeltaArgs {
 // rows of S in registers, NSL row slices of a column in neighbouring lanes; kRecTile tokens staged with cp.async two stages
 // deep).  Per token one pass over the registers decays S and accumulates both S^T k and S^T q of the DECAYED state; after the
 // lanes' partial sums meet (shuffles) u = beta (v - S^T k) is known, a second pass adds k u^T, and the read-out of the updated
-// state is  S^T q + u (k . q)  — no third pass.
-template <int NPT, int NSL, int PP>
+// state is  S^T q + u (k . q)  — no third pass.  HEADG: one decay per head (a scalar per token) instead of one per key channel.
+template <int NPT, int NSL, int PP, bool HEADG>
 __global__ void __launch_bounds__(512) gated_delta_kernel(const DeltaArgs a, int pb, int vec) {
   extern __shared__ __align__(16) float sm[];
   constexpr int SL = NPT + 4, DKP = SL * NSL;
   const int pbp = (pb + 3) & ~3;
-  const int stage = kRecTile * (3 * DKP + pbp + 4);
+  const int stage = kRecTile * ((HEADG ? 2 : 3) * DKP + pbp + 4);
   const int h = blockIdx.x, s = blockIdx.y, p0 = blockIdx.z * pb;
   const int tid = threadIdx.x, ns = tid % NSL, pl = tid / NSL, p = p0 + pl, half = (pb + PP - 1) / PP;
   bool live[PP];
@@ -220,9 +229,10 @@ __global__ void __launch_bounds__(512) gated_delta_kernel(const DeltaArgs a, int
   auto issue = [&](int tb, int buf) {
     float* ks = sm + buf * stage;
     float* qs = ks + kRecTile * DKP;
-    float* gs = qs + kRecTile * DKP;
-    float* vs = gs + kRecTile * DKP;
+    float* gs = qs + kRecTile * DKP;               // per-channel decays only
+    float* vs = gs + (HEADG ? 0 : kRecTile * DKP);
     float* bs = vs + kRecTile * pbp;
+    float* ds = bs + kRecTile;                     // per-head decays only
     const int cnt = min(kRecTile, t1 - tb);
     if (vec) {
       const int kch = a.dk / 4, vch = ncol / 4;
@@ -232,7 +242,7 @@ __global__ void __launch_bounds__(512) gated_delta_kernel(const DeltaArgs a, int
         const int dst = tt * DKP + (c * 4 / NPT) * SL + (c * 4) % NPT;
         cp_async_16(smem_u32(ks + dst), a.k + t * a.ldk + static_cast<int64_t>(g) * a.dk + c * 4, 16);
         cp_async_16(smem_u32(qs + dst), a.q + t * a.ldq + static_cast<int64_t>(g) * a.dk + c * 4, 16);
-        cp_async_16(smem_u32(gs + dst), a.decay + t * a.ldd + static_cast<int64_t>(h) * a.dk + c * 4, 16);
+        if (!HEADG) cp_async_16(smem_u32(gs + dst), a.decay + t * a.ldd + static_cast<int64_t>(h) * a.dk + c * 4, 16);
       }
       for (int e = tid; e < cnt * vch; e += blockDim.x) {
         const int tt = e / vch, c = e - tt * vch;
@@ -245,14 +255,17 @@ __global__ void __launch_bounds__(512) gated_delta_kernel(const DeltaArgs a, int
         const int dst = tt * DKP + (n / NPT) * SL + n % NPT;
         cp_async_4(smem_u32(ks + dst), a.k + t * a.ldk + static_cast<int64_t>(g) * a.dk + n);
         cp_async_4(smem_u32(qs + dst), a.q + t * a.ldq + static_cast<int64_t>(g) * a.dk + n);
-        cp_async_4(smem_u32(gs + dst), a.decay + t * a.ldd + static_cast<int64_t>(h) * a.dk + n);
+        if (!HEADG) cp_async_4(smem_u32(gs + dst), a.decay + t * a.ldd + static_cast<int64_t>(h) * a.dk + n);
       }
       for (int e = tid; e < cnt * ncol; e += blockDim.x) {
         const int tt = e / ncol, c = e - tt * ncol;
         cp_async_4(smem_u32(vs + tt * pbp + c), a.v + static_cast<int64_t>(tb + tt) * a.ldv + static_cast<int64_t>(h) * a.dv + p0 + c);
       }
     }
-    if (tid < cnt) cp_async_4(smem_u32(bs + tid), a.beta + (tb + tid) * a.ldb + h);
+    if (tid < cnt) {
+      cp_async_4(smem_u32(bs + tid), a.beta + (tb + tid) * a.ldb + h);
+      if (HEADG) cp_async_4(smem_u32(ds + tid), a.decay + (tb + tid) * a.ldd + h);
+    }
     cp_async_commit();
   };
   issue(t0, 0);
@@ -274,10 +287,11 @@ __global__ void __launch_bounds__(512) gated_delta_kernel(const DeltaArgs a, int
     const float* ks = sm + buf * stage;
     const float* qs = ks + kRecTile * DKP;
     const float* gs = qs + kRecTile * DKP;
-    const float* vs = gs + kRecTile * DKP;
+    const float* vs = gs + (HEADG ? 0 : kRecTile * DKP);
     const float* bs = vs + kRecTile * pbp;
+    const float* ds = bs + kRecTile;
     for (int tt = 0; tt < cnt; ++tt) {
-      const float bt = bs[tt];
+      const float bt = bs[tt], dt = HEADG ? ds[tt] : 0.f;
       float xv[PP], rk[PP], rq[PP], kq = 0.f;
 #pragma unroll
       for (int j = 0; j < PP; ++j) { xv[j] = vs[tt * pbp + (live[j] ? pl + j * half : 0)]; rk[j] = 0.f; rq[j] = 0.f; }
@@ -286,7 +300,7 @@ __global__ void __launch_bounds__(512) gated_delta_kernel(const DeltaArgs a, int
       const float4* gr = reinterpret_cast<const float4*>(gs + tt * DKP + ns * SL);
 #pragma unroll
       for (int i = 0; i < NPT / 4; ++i) {
-        const float4 k4 = kr[i], q4 = qr[i], g4 = gr[i];
+        const float4 k4 = kr[i], q4 = qr[i], g4 = HEADG ? make_float4(dt, dt, dt, dt) : gr[i];
         kq = fmaf(k4.x, q4.x, fmaf(k4.y, q4.y, fmaf(k4.z, q4.z, fmaf(k4.w, q4.w, kq))));
 #pragma unroll
         for (int j = 0; j < PP; ++j) {
@@ -335,6 +349,7 @@ struct DeltaPrepArgs {
   float *q, *k, *beta, *decay; int64_t ldq, ldk, ldb, ldd;
   const float *a_log, *dt_bias;
   int heads, groups, dk; float q_scale, unit_eps;
+  int head_decay;   // decay, dt_bias: one value per head instead of one per key channel
 };
 
 // CTA per token: the warps take the 2 * groups vectors of q and k (unit length; q also scaled), then all threads the
@@ -354,12 +369,12 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(const DeltaPrepArgs 
     float* b = a.beta + t * a.ldb + h;
     *b = 1.0f / (1.0f + expf(-*b));
   }
-  const int hd = a.heads * a.dk;
+  const int hd = a.head_decay ? a.heads : a.heads * a.dk, per = a.head_decay ? 1 : a.dk;
   for (int e = threadIdx.x; e < hd; e += blockDim.x) {
     float* d = a.decay + t * a.ldd + e;
     const float x = *d + a.dt_bias[e];
     const float dt = x > 20.f ? x : log1pf(expf(x));
-    *d = expf(-expf(a.a_log[e / a.dk]) * dt);
+    *d = expf(-expf(a.a_log[e / per]) * dt);
   }
 }
 
@@ -393,12 +408,57 @@ __global__ void __launch_bounds__(256) delta_prepare_vec_kernel(const DeltaPrepA
     const float dt = x > 20.f ? x : log1pf(expf(x));
     return expf(-ea * dt);
   };
+  if (a.head_decay) {
+    for (int h = threadIdx.x; h < a.heads; h += blockDim.x) {
+      float* d = a.decay + t * a.ldd + h;
+      *d = decay(*d, a.dt_bias[h], expf(a.a_log[h]));
+    }
+    return;
+  }
   const int hd4 = a.heads * nv;
   float4* d = reinterpret_cast<float4*>(a.decay + t * a.ldd);
   for (int e = threadIdx.x; e < hd4; e += blockDim.x) {
     const float ea = expf(a.a_log[e / nv]);
     const float4 raw = d[e], b = reinterpret_cast<const float4*>(a.dt_bias)[e];
     d[e] = make_float4(decay(raw.x, b.x, ea), decay(raw.y, b.y, ea), decay(raw.z, b.z, ea), decay(raw.w, b.w, ea));
+  }
+}
+
+// out[t, c] = sigmoid(sum_r w2[r, c] x[t, r] + b[c])^(1 / tau) = exp(log sigmoid(z) / tau): the second step of a two-step projection,
+// its bias and the decay in one pass, all f32.  CTA = 16 tokens x 128 channels: the tokens' inner values in shared memory,
+// a thread per channel (w2 is stored [rank, channels]: coalesced), every weight read serves 16 tokens.
+constexpr int kLrTok = 16, kLrRank = 64;
+__global__ void __launch_bounds__(128) low_rank_decay_kernel(float* __restrict__ out, int64_t ldo, const float* __restrict__ x, int64_t ldx,
+                                                             const float* __restrict__ w2, const float* __restrict__ bias, int n, int rank,
+                                                             int channels, float inv_tau) {
+  __shared__ float xs[kLrRank][kLrTok];
+  const int c = blockIdx.x * 128 + threadIdx.x, t0 = blockIdx.y * kLrTok, cnt = min(kLrTok, n - t0);
+  float acc[kLrTok];
+#pragma unroll
+  for (int t = 0; t < kLrTok; ++t) acc[t] = 0.f;
+  for (int r0 = 0; r0 < rank; r0 += kLrRank) {
+    const int rc = min(kLrRank, rank - r0);
+    __syncthreads();
+    for (int e = threadIdx.x; e < kLrTok * rc; e += 128) {
+      const int t = e / rc, r = e - t * rc;
+      xs[r][t] = t < cnt ? x[(t0 + t) * ldx + r0 + r] : 0.f;
+    }
+    __syncthreads();
+    if (c < channels) {
+      for (int r = 0; r < rc; ++r) {
+        const float w = w2[static_cast<int64_t>(r0 + r) * channels + c];
+#pragma unroll
+        for (int t = 0; t < kLrTok; ++t) acc[t] = fmaf(w, xs[r][t], acc[t]);
+      }
+    }
+  }
+  if (c >= channels) return;
+  const float b = bias ? bias[c] : 0.f;
+#pragma unroll
+  for (int t = 0; t < kLrTok; ++t) {
+    if (t >= cnt) break;
+    const float z = acc[t] + b;
+    out[(t0 + t) * ldo + c] = expf((fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * inv_tau);
   }
 }
 
@@ -672,41 +732,73 @@ inline unsigned grid_for(int64_t total) {
   return static_cast<unsigned>(b > cap ? cap : (b < 1 ? 1 : b));
 }
 
-template <int NPT, int NSL, int PP>
-int launch_recurrence(const RecArgs& a, int n_seqs, cudaStream_t st) {
+template <int NPT, int NSL, int PP, bool CHD>
+int launch_recurrence_as(const RecArgs& a, int n_seqs, cudaStream_t st) {
   int pb = a.dv;                                  // columns per CTA
   const int max_pb = 512 / NSL * PP;
   if (pb > max_pb) pb = max_pb;
   // more CTAs when few (sequence, head) pairs would leave SMs idle: split the columns (each column is independent)
   while (pb > 32 && static_cast<int64_t>(a.heads) * n_seqs * ((a.dv + pb - 1) / pb) < sm_count() && pb % 2 == 0) pb /= 2;
   const int threads = (((pb + PP - 1) / PP * NSL + 31) / 32) * 32;
-  const size_t smem = 2 * static_cast<size_t>(kRecTile) * (2 * (NPT + 4) * NSL + ((pb + 3) & ~3) + 2) * sizeof(float);
+  const size_t smem = 2 * static_cast<size_t>(kRecTile) * ((CHD ? 3 : 2) * (NPT + 4) * NSL + ((pb + 3) & ~3) + 2) * sizeof(float);
   dim3 grid(a.heads, n_seqs, (a.dv + pb - 1) / pb);
-  if (smem > 48 * 1024) NVLLM_CUDA(cudaFuncSetAttribute(linear_recurrence_kernel<NPT, NSL, PP>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
+  if (smem > 48 * 1024) NVLLM_CUDA(cudaFuncSetAttribute(linear_recurrence_kernel<NPT, NSL, PP, CHD>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
   // 16-byte copies when every staged row starts and ends on a 16-byte boundary
   const int vec = a.dk % 4 == 0 && a.dv % 4 == 0 && pb % 4 == 0 && a.ldq % 4 == 0 && a.ldk % 4 == 0 && a.ldv % 4 == 0 && aligned16(a.q) &&
-                  aligned16(a.k) && aligned16(a.v);
-  linear_recurrence_kernel<NPT, NSL, PP><<<grid, threads, smem, st>>>(a, pb, vec);
+                  aligned16(a.k) && aligned16(a.v) && (!CHD || (a.decay_ld % 4 == 0 && aligned16(a.decay)));
+  linear_recurrence_kernel<NPT, NSL, PP, CHD><<<grid, threads, smem, st>>>(a, pb, vec);
   NVLLM_LAUNCH_CHECK("linear_recurrence_kernel");
   return 0;
 }
 
+template <bool CHD>
+int launch_recurrence(const RecArgs& a, int n_seqs, cudaStream_t st) {
+  if (a.dk <= 16) return launch_recurrence_as<16, 1, 2, CHD>(a, n_seqs, st);
+  if (a.dk <= 32) return launch_recurrence_as<32, 1, 2, CHD>(a, n_seqs, st);
+  if (a.dk <= 64) return launch_recurrence_as<32, 2, 2, CHD>(a, n_seqs, st);
+  if (a.dk <= 128) return launch_recurrence_as<32, 4, 2, CHD>(a, n_seqs, st);
+  if (a.dk <= 256) return launch_recurrence_as<32, 8, 2, CHD>(a, n_seqs, st);
+  return launch_recurrence_as<32, 16, 2, CHD>(a, n_seqs, st);
+}
 
-template <int NPT, int NSL, int PP>
-int launch_delta(const DeltaArgs& a, int n_seqs, cudaStream_t st) {
+template <int NPT, int NSL, int PP, bool HEADG>
+int launch_delta_as(const DeltaArgs& a, int n_seqs, cudaStream_t st) {
   int pb = a.dv;                                  // columns per CTA
   const int max_pb = 512 / NSL * PP;
   if (pb > max_pb) pb = max_pb;
   while (pb > 32 && static_cast<int64_t>(a.heads) * n_seqs * ((a.dv + pb - 1) / pb) < sm_count() && pb % 2 == 0) pb /= 2;
   const int threads = (((pb + PP - 1) / PP * NSL + 31) / 32) * 32;
-  const size_t smem = 2 * static_cast<size_t>(kRecTile) * (3 * (NPT + 4) * NSL + ((pb + 3) & ~3) + 4) * sizeof(float);
+  const size_t smem = 2 * static_cast<size_t>(kRecTile) * ((HEADG ? 2 : 3) * (NPT + 4) * NSL + ((pb + 3) & ~3) + 4) * sizeof(float);
   dim3 grid(a.heads, n_seqs, (a.dv + pb - 1) / pb);
-  if (smem > 48 * 1024) NVLLM_CUDA(cudaFuncSetAttribute(gated_delta_kernel<NPT, NSL, PP>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
-  const int vec = a.dk % 4 == 0 && a.dv % 4 == 0 && pb % 4 == 0 && a.ldq % 4 == 0 && a.ldk % 4 == 0 && a.ldv % 4 == 0 && a.ldd % 4 == 0 &&
-                  aligned16(a.q) && aligned16(a.k) && aligned16(a.v) && aligned16(a.decay);
-  gated_delta_kernel<NPT, NSL, PP><<<grid, threads, smem, st>>>(a, pb, vec);
+  if (smem > 48 * 1024) NVLLM_CUDA(cudaFuncSetAttribute(gated_delta_kernel<NPT, NSL, PP, HEADG>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
+  const int vec = a.dk % 4 == 0 && a.dv % 4 == 0 && pb % 4 == 0 && a.ldq % 4 == 0 && a.ldk % 4 == 0 && a.ldv % 4 == 0 &&
+                  aligned16(a.q) && aligned16(a.k) && aligned16(a.v) && (HEADG || (a.ldd % 4 == 0 && aligned16(a.decay)));
+  gated_delta_kernel<NPT, NSL, PP, HEADG><<<grid, threads, smem, st>>>(a, pb, vec);
   NVLLM_LAUNCH_CHECK("gated_delta_kernel");
   return 0;
+}
+
+template <bool HEADG>
+int launch_delta(const DeltaArgs& a, int n_seqs, cudaStream_t st) {
+  if (a.dk <= 16) return launch_delta_as<16, 1, 2, HEADG>(a, n_seqs, st);
+  if (a.dk <= 32) return launch_delta_as<32, 1, 2, HEADG>(a, n_seqs, st);
+  if (a.dk <= 64) return launch_delta_as<32, 2, 2, HEADG>(a, n_seqs, st);
+  if (a.dk <= 128) {
+    switch (knobs().delta_cfg) {   // A/B: how a column's rows are split over lanes and how many columns a thread holds
+      case 1: return launch_delta_as<16, 8, 2, HEADG>(a, n_seqs, st);
+      case 2: return launch_delta_as<32, 4, 1, HEADG>(a, n_seqs, st);
+      case 3: return launch_delta_as<16, 8, 1, HEADG>(a, n_seqs, st);
+      case 4: return launch_delta_as<8, 16, 2, HEADG>(a, n_seqs, st);
+      case 5: return launch_delta_as<16, 8, 4, HEADG>(a, n_seqs, st);
+      default:
+        // few (head, sequence) pairs: twice the lanes per column keep more warps in flight (one long prompt: 1.35 vs 2.03 ms
+        // for 4096 tokens of 16 heads); otherwise the wider slices win (8 x 1024 tokens: 0.79 vs 0.77 ms, single tokens 41 vs 57 us)
+        if (static_cast<int64_t>(a.heads) * n_seqs * 2 <= sm_count()) return launch_delta_as<16, 8, 2, HEADG>(a, n_seqs, st);
+        return launch_delta_as<32, 4, 2, HEADG>(a, n_seqs, st);
+    }
+  }
+  if (a.dk <= 256) return launch_delta_as<32, 8, 2, HEADG>(a, n_seqs, st);
+  return launch_delta_as<32, 16, 2, HEADG>(a, n_seqs, st);
 }
 
 }  // namespace
@@ -714,21 +806,49 @@ int launch_delta(const DeltaArgs& a, int n_seqs, cudaStream_t st) {
 
 using namespace nvllm;
 
-extern "C" int nvllm_delta_prepare(float* q, int64_t ldq, float* k, int64_t ldk, float* beta, int64_t ldb, float* decay, int64_t ldd,
-                                   const float* a_log, const float* dt_bias, int32_t n, int32_t heads, int32_t groups, int32_t dk,
-                                   float q_scale, float unit_eps, void* stream) {
+namespace {
+int delta_prepare(float* q, int64_t ldq, float* k, int64_t ldk, float* beta, int64_t ldb, float* decay, int64_t ldd, const float* a_log,
+                  const float* dt_bias, int32_t n, int32_t heads, int32_t groups, int32_t dk, float q_scale, float unit_eps, int head_decay,
+                  void* stream) {
   NVLLM_CHECK_ARG(n >= 0 && heads > 0 && groups > 0 && dk > 0 && ldq >= static_cast<int64_t>(groups) * dk && ldk >= static_cast<int64_t>(groups) * dk &&
-                      ldb >= heads && ldd >= static_cast<int64_t>(heads) * dk, NVLLM_ERR_ARG, "delta_prepare: sizes");
+                      ldb >= heads && ldd >= static_cast<int64_t>(heads) * (head_decay ? 1 : dk), NVLLM_ERR_ARG, "delta_prepare: sizes");
   if (n == 0) return 0;
   NVLLM_CHECK_ARG(q && k && beta && decay && a_log && dt_bias, NVLLM_ERR_ARG, "delta_prepare: NULL");
-  const DeltaPrepArgs a{q, k, beta, decay, ldq, ldk, ldb, ldd, a_log, dt_bias, heads, groups, dk, q_scale, unit_eps};
-  if (dk % 4 == 0 && dk <= 512 && ldq % 4 == 0 && ldk % 4 == 0 && ldd % 4 == 0 && aligned16(q) && aligned16(k) && aligned16(decay) && aligned16(dt_bias)) {
+  const DeltaPrepArgs a{q, k, beta, decay, ldq, ldk, ldb, ldd, a_log, dt_bias, heads, groups, dk, q_scale, unit_eps, head_decay};
+  if (dk % 4 == 0 && dk <= 512 && ldq % 4 == 0 && ldk % 4 == 0 && aligned16(q) && aligned16(k) &&
+      (head_decay || (ldd % 4 == 0 && aligned16(decay) && aligned16(dt_bias)))) {
     delta_prepare_vec_kernel<<<n, 256, 0, static_cast<cudaStream_t>(stream)>>>(a);
     NVLLM_LAUNCH_CHECK("delta_prepare_vec_kernel");
     return 0;
   }
   delta_prepare_kernel<<<n, 128, 0, static_cast<cudaStream_t>(stream)>>>(a);
   NVLLM_LAUNCH_CHECK("delta_prepare_kernel");
+  return 0;
+}
+
+}  // namespace
+
+extern "C" int nvllm_delta_prepare(float* q, int64_t ldq, float* k, int64_t ldk, float* beta, int64_t ldb, float* decay, int64_t ldd,
+                                   const float* a_log, const float* dt_bias, int32_t n, int32_t heads, int32_t groups, int32_t dk,
+                                   float q_scale, float unit_eps, void* stream) {
+  return delta_prepare(q, ldq, k, ldk, beta, ldb, decay, ldd, a_log, dt_bias, n, heads, groups, dk, q_scale, unit_eps, 0, stream);
+}
+
+extern "C" int nvllm_head_delta_prepare(float* q, int64_t ldq, float* k, int64_t ldk, float* beta, int64_t ldb, float* decay, int64_t ldd,
+                                        const float* a_log, const float* dt_bias, int32_t n, int32_t heads, int32_t groups, int32_t dk,
+                                        float q_scale, float unit_eps, void* stream) {
+  return delta_prepare(q, ldq, k, ldk, beta, ldb, decay, ldd, a_log, dt_bias, n, heads, groups, dk, q_scale, unit_eps, 1, stream);
+}
+
+extern "C" int nvllm_low_rank_decay(float* out, int64_t ldo, const float* x, int64_t ldx, const float* w2, const float* bias, int32_t n,
+                                    int32_t rank, int32_t channels, float tau, void* stream) {
+  NVLLM_CHECK_ARG(n >= 0 && rank > 0 && channels > 0 && ldx >= rank && ldo >= channels && tau > 0.f, NVLLM_ERR_ARG,
+                  "low_rank_decay: n=%d rank=%d channels=%d tau=%g", n, rank, channels, tau);
+  if (n == 0) return 0;
+  NVLLM_CHECK_ARG(out && x && w2, NVLLM_ERR_ARG, "low_rank_decay: NULL");
+  dim3 grid((channels + 127) / 128, (n + kLrTok - 1) / kLrTok);
+  low_rank_decay_kernel<<<grid, 128, 0, static_cast<cudaStream_t>(stream)>>>(out, ldo, x, ldx, w2, bias, n, rank, channels, 1.0f / tau);
+  NVLLM_LAUNCH_CHECK("low_rank_decay_kernel");
   return 0;
 }
 
@@ -742,25 +862,32 @@ extern "C" int nvllm_gated_delta_recurrence(float* y, int64_t ldy, const float* 
   NVLLM_CHECK_ARG(y && q && k && v && decay && beta && state && seq_slot && cu_tokens && positions, NVLLM_ERR_ARG, "gated_delta_recurrence: NULL");
   DeltaArgs a{y, ldy, q, k, v, ldq, ldk, ldv, heads / groups, decay, ldd, beta, ldb, state, seq_slot, cu_tokens, positions, heads, dk, dv};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (dk <= 16) return launch_delta<16, 1, 2>(a, n_seqs, st);
-  if (dk <= 32) return launch_delta<32, 1, 2>(a, n_seqs, st);
-  if (dk <= 64) return launch_delta<32, 2, 2>(a, n_seqs, st);
-  if (dk <= 128) {
-    switch (knobs().delta_cfg) {   // A/B: how a column's rows are split over lanes and how many columns a thread holds
-      case 1: return launch_delta<16, 8, 2>(a, n_seqs, st);
-      case 2: return launch_delta<32, 4, 1>(a, n_seqs, st);
-      case 3: return launch_delta<16, 8, 1>(a, n_seqs, st);
-      case 4: return launch_delta<8, 16, 2>(a, n_seqs, st);
-      case 5: return launch_delta<16, 8, 4>(a, n_seqs, st);
-      default:
-        // few (head, sequence) pairs: twice the lanes per column keep more warps in flight (one long prompt: 1.35 vs 2.03 ms
-        // for 4096 tokens of 16 heads); otherwise the wider slices win (8 x 1024 tokens: 0.79 vs 0.77 ms, single tokens 41 vs 57 us)
-        if (static_cast<int64_t>(heads) * n_seqs * 2 <= sm_count()) return launch_delta<16, 8, 2>(a, n_seqs, st);
-        return launch_delta<32, 4, 2>(a, n_seqs, st);
-    }
-  }
-  if (dk <= 256) return launch_delta<32, 8, 2>(a, n_seqs, st);
-  return launch_delta<32, 16, 2>(a, n_seqs, st);
+  return launch_delta<false>(a, n_seqs, st);
+}
+
+extern "C" int nvllm_head_delta_recurrence(float* y, int64_t ldy, const float* q, int64_t ldq, const float* k, int64_t ldk, const float* v,
+                                           int64_t ldv, const float* decay, int64_t ldd, const float* beta, int64_t ldb, float* state,
+                                           const int32_t* seq_slot, const int32_t* cu_tokens, const int64_t* positions, int32_t n_seqs,
+                                           int32_t heads, int32_t groups, int32_t dk, int32_t dv, void* stream) {
+  NVLLM_CHECK_ARG(n_seqs >= 0 && heads > 0 && groups > 0 && heads % groups == 0 && dk > 0 && dk <= 512 && dv > 0, NVLLM_ERR_ARG,
+                  "head_delta_recurrence: seqs=%d heads=%d groups=%d dk=%d (<= 512) dv=%d", n_seqs, heads, groups, dk, dv);
+  if (n_seqs == 0) return 0;
+  NVLLM_CHECK_ARG(y && q && k && v && decay && beta && state && seq_slot && cu_tokens && positions, NVLLM_ERR_ARG, "head_delta_recurrence: NULL");
+  const DeltaArgs a{y, ldy, q, k, v, ldq, ldk, ldv, heads / groups, decay, ldd, beta, ldb, state, seq_slot, cu_tokens, positions, heads, dk, dv};
+  return launch_delta<true>(a, n_seqs, static_cast<cudaStream_t>(stream));
+}
+
+extern "C" int nvllm_channel_recurrence(float* y, int64_t ldy, const float* q, int64_t ldq, const float* k, int64_t ldk, const float* v,
+                                        int64_t ldv, const float* decay, int64_t ldd, float q_scale, float* state, const int32_t* seq_slot,
+                                        const int32_t* cu_tokens, const int64_t* positions, int32_t n_seqs, int32_t heads, int32_t groups,
+                                        int32_t dk, int32_t dv, void* stream) {
+  NVLLM_CHECK_ARG(n_seqs >= 0 && heads > 0 && groups > 0 && heads % groups == 0 && dk > 0 && dk <= 512 && dv > 0, NVLLM_ERR_ARG,
+                  "channel_recurrence: seqs=%d heads=%d groups=%d dk=%d (<= 512) dv=%d", n_seqs, heads, groups, dk, dv);
+  if (n_seqs == 0) return 0;
+  NVLLM_CHECK_ARG(y && q && k && v && decay && state && seq_slot && cu_tokens && positions, NVLLM_ERR_ARG, "channel_recurrence: NULL");
+  const RecArgs a{y, ldy, q, k, v, ldq, ldk, ldv, heads / groups, decay, ldd, nullptr, 0, nullptr, state, seq_slot, cu_tokens, positions,
+                  heads, dk, dv, q_scale};
+  return launch_recurrence<true>(a, n_seqs, static_cast<cudaStream_t>(stream));
 }
 
 extern "C" int nvllm_linear_recurrence(float* y, int64_t ldy, const float* q, int64_t ldq, const float* k, int64_t ldk, const float* v,
@@ -773,14 +900,9 @@ extern "C" int nvllm_linear_recurrence(float* y, int64_t ldy, const float* q, in
   if (n_seqs == 0) return 0;
   NVLLM_CHECK_ARG(y && q && k && v && decay && state && seq_slot && cu_tokens && positions, NVLLM_ERR_ARG, "linear_recurrence: NULL");
   RecArgs a{y, ldy, q, k, v, ldq, ldk, ldv, heads / groups, decay, decay_per_token ? heads : 0, step, step_per_token ? heads : 0,
-            skip, state, seq_slot, cu_tokens, positions, heads, dk, dv};
+            skip, state, seq_slot, cu_tokens, positions, heads, dk, dv, 1.0f};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (dk <= 16) return launch_recurrence<16, 1, 2>(a, n_seqs, st);
-  if (dk <= 32) return launch_recurrence<32, 1, 2>(a, n_seqs, st);
-  if (dk <= 64) return launch_recurrence<32, 2, 2>(a, n_seqs, st);
-  if (dk <= 128) return launch_recurrence<32, 4, 2>(a, n_seqs, st);
-  if (dk <= 256) return launch_recurrence<32, 8, 2>(a, n_seqs, st);
-  return launch_recurrence<32, 16, 2>(a, n_seqs, st);
+  return launch_recurrence<false>(a, n_seqs, st);
 }
 
 extern "C" int nvllm_causal_conv(float* out, int64_t ldo, const float* in, int64_t ldi, const float* w, const float* bias, float* state,

@@ -5,6 +5,8 @@
 //                             (pre_w == NULL: out = h, for blocks whose sublayers read the stream without a norm)
 //                             (the sublayer's output norm, the residual add and the next sublayer's input norm in one pass over
 //                             the row, as nvllm_dyt_residual_norm does for Dynamic Tanh models)
+//   nvllm_rms_sum_norm        the step of a block that norms the SUM (post-norm of the classic transformer, weighted skip):
+//                                 h = rms(alpha * h + y) * w;   out = h, or rms(h) * last_w behind the last layer
 //   nvllm_rms_norm_rows       rows of an f32 matrix, RMS-normed and weighted, written in the operand type to rows of a
 //                             destination chosen by a map (a paged cache's slots) or in place of order
 //   nvllm_embedding_stream    h[t] = table[id_t] * scale as f32 and, in the same pass, in the operand type
@@ -135,6 +137,99 @@ __global__ void __launch_bounds__(256) rms_residual_norm_vec_kernel(TO* __restri
       else reinterpret_cast<float4*>(reinterpret_cast<float*>(out) + base)[c] = o;
     }
   }
+}
+
+// h = rms(alpha * h + y) * w;  out = last_w ? rms(h) * last_w : h.  CTA per row, the row in shared memory between the passes.
+template <typename TO>
+__global__ void __launch_bounds__(256) rms_sum_norm_kernel(TO* __restrict__ out, float* __restrict__ h, const void* __restrict__ y, int y_dt, float alpha,
+                                                           const float* __restrict__ w, const float* __restrict__ last_w, int hidden, float eps) {
+  extern __shared__ float row[];
+  __shared__ float red[8];
+  const int64_t base = static_cast<int64_t>(blockIdx.x) * hidden;
+  float sq = 0.f;
+  for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
+    const float v = fmaf(alpha, h[base + c], ld_any(y, y_dt, base + c));
+    row[c] = v;
+    sq = fmaf(v, v, sq);
+  }
+  const float r = 1.0f / sqrtf(block_sum(sq, red) / hidden + eps);
+  sq = 0.f;
+  for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
+    const float v = row[c] * r * w[c];
+    h[base + c] = v;
+    if (last_w == nullptr) st_as(out, base + c, v);
+    row[c] = v;
+    sq = fmaf(v, v, sq);
+  }
+  if (last_w == nullptr) return;
+  const float r2 = 1.0f / sqrtf(block_sum(sq, red) / hidden + eps);
+  for (int c = threadIdx.x; c < hidden; c += blockDim.x) st_as(out, base + c, row[c] * r2 * last_w[c]);
+}
+
+// The same for rows of up to 1024 NK values in 16-byte vectors, the row in registers (one global pass).
+template <int NK, typename TY, typename TO>
+__global__ void __launch_bounds__(256) rms_sum_norm_vec_kernel(TO* __restrict__ out, float* __restrict__ h, const TY* __restrict__ y, float alpha,
+                                                               const float* __restrict__ w, const float* __restrict__ last_w, int hidden, float eps) {
+  __shared__ float red[8];
+  const int nv = hidden / 4;
+  const int64_t base = static_cast<int64_t>(blockIdx.x) * hidden;
+  float4* hr = reinterpret_cast<float4*>(h + base);
+  float4 v[NK];
+  float sq = 0.f;
+#pragma unroll
+  for (int k = 0; k < NK; ++k) {
+    const int c = threadIdx.x + 256 * k;
+    if (c < nv) {
+      float4 yv;
+      if (sizeof(TY) == 2) {
+        const uint2 u = reinterpret_cast<const uint2*>(reinterpret_cast<const bf16*>(y) + base)[c];
+        yv = make_float4(bf16_lo(u.x), bf16_hi(u.x), bf16_lo(u.y), bf16_hi(u.y));
+      } else {
+        yv = reinterpret_cast<const float4*>(reinterpret_cast<const float*>(y) + base)[c];
+      }
+      const float4 hv = hr[c];
+      v[k] = make_float4(fmaf(alpha, hv.x, yv.x), fmaf(alpha, hv.y, yv.y), fmaf(alpha, hv.z, yv.z), fmaf(alpha, hv.w, yv.w));
+      sq += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+    }
+  }
+  auto put = [&](int c, const float4& o) {
+    if (sizeof(TO) == 2) reinterpret_cast<uint2*>(reinterpret_cast<bf16*>(out) + base)[c] = make_uint2(pack_bf16x2(o.x, o.y), pack_bf16x2(o.z, o.w));
+    else reinterpret_cast<float4*>(reinterpret_cast<float*>(out) + base)[c] = o;
+  };
+  const float r = 1.0f / sqrtf(block_sum(sq, red) / hidden + eps);
+  sq = 0.f;
+#pragma unroll
+  for (int k = 0; k < NK; ++k) {
+    const int c = threadIdx.x + 256 * k;
+    if (c < nv) {
+      const float4 ww = reinterpret_cast<const float4*>(w)[c];
+      v[k] = make_float4(v[k].x * r * ww.x, v[k].y * r * ww.y, v[k].z * r * ww.z, v[k].w * r * ww.w);
+      hr[c] = v[k];
+      if (last_w == nullptr) put(c, v[k]);
+      sq += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+    }
+  }
+  if (last_w == nullptr) return;
+  const float r2 = 1.0f / sqrtf(block_sum(sq, red) / hidden + eps);
+#pragma unroll
+  for (int k = 0; k < NK; ++k) {
+    const int c = threadIdx.x + 256 * k;
+    if (c < nv) {
+      const float4 ww = reinterpret_cast<const float4*>(last_w)[c];
+      put(c, make_float4(v[k].x * r2 * ww.x, v[k].y * r2 * ww.y, v[k].z * r2 * ww.z, v[k].w * r2 * ww.w));
+    }
+  }
+}
+
+template <typename TY, typename TO>
+int launch_sum_norm_vec(void* out, float* h, const void* y, float alpha, const float* w, const float* last_w, int n, int hidden, float eps, cudaStream_t st) {
+  TO* o = static_cast<TO*>(out);
+  const TY* yy = static_cast<const TY*>(y);
+  if (hidden <= 2048) rms_sum_norm_vec_kernel<2, TY, TO><<<n, 256, 0, st>>>(o, h, yy, alpha, w, last_w, hidden, eps);
+  else if (hidden <= 4096) rms_sum_norm_vec_kernel<4, TY, TO><<<n, 256, 0, st>>>(o, h, yy, alpha, w, last_w, hidden, eps);
+  else rms_sum_norm_vec_kernel<8, TY, TO><<<n, 256, 0, st>>>(o, h, yy, alpha, w, last_w, hidden, eps);
+  NVLLM_LAUNCH_CHECK("rms_sum_norm_vec_kernel");
+  return 0;
 }
 
 // One warp per row.
@@ -269,6 +364,33 @@ extern "C" int nvllm_rms_residual_norm(void* out, float* h, const void* y, int32
     rms_residual_norm_kernel<float><<<n, 256, smem, st>>>(static_cast<float*>(out), h, y, y_dtype, post_w, pre_w, hidden, eps);
   }
   NVLLM_LAUNCH_CHECK("rms_residual_norm_kernel");
+  return 0;
+}
+
+extern "C" int nvllm_rms_sum_norm(void* out, float* h, const void* y, int32_t y_dtype, float alpha, const float* w, const float* last_w,
+                                  int32_t n, int32_t hidden, float eps, int32_t out_dtype, void* stream) {
+  NVLLM_CHECK_ARG(n >= 0 && hidden > 0 && hidden <= 48 * 1024, NVLLM_ERR_ARG, "rms_sum_norm: n=%d hidden=%d (<= 49152)", n, hidden);
+  NVLLM_CHECK_ARG((out_dtype == NVLLM_BF16 || out_dtype == NVLLM_F32) && (y_dtype == NVLLM_BF16 || y_dtype == NVLLM_F32), NVLLM_ERR_DTYPE,
+                  "rms_sum_norm: dtype %d / %d", y_dtype, out_dtype);
+  if (n == 0) return 0;
+  NVLLM_CHECK_ARG(out && h && y && w, NVLLM_ERR_ARG, "rms_sum_norm: NULL");
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const bool yb = y_dtype == NVLLM_BF16, ob = out_dtype == NVLLM_BF16;
+  if (hidden % 4 == 0 && hidden <= 8192 && aligned16(h) && aligned16(y) && aligned16(out) && aligned16(w) && aligned16(last_w)) {
+    if (yb && ob) return launch_sum_norm_vec<bf16, bf16>(out, h, y, alpha, w, last_w, n, hidden, eps, st);
+    if (yb) return launch_sum_norm_vec<bf16, float>(out, h, y, alpha, w, last_w, n, hidden, eps, st);
+    if (ob) return launch_sum_norm_vec<float, bf16>(out, h, y, alpha, w, last_w, n, hidden, eps, st);
+    return launch_sum_norm_vec<float, float>(out, h, y, alpha, w, last_w, n, hidden, eps, st);
+  }
+  const size_t smem = static_cast<size_t>(hidden) * sizeof(float);
+  if (ob) {
+    NVLLM_SMEM_ATTR_ONCE(rms_sum_norm_kernel<bf16>, 192 * 1024);
+    rms_sum_norm_kernel<bf16><<<n, 256, smem, st>>>(static_cast<bf16*>(out), h, y, y_dtype, alpha, w, last_w, hidden, eps);
+  } else {
+    NVLLM_SMEM_ATTR_ONCE(rms_sum_norm_kernel<float>, 192 * 1024);
+    rms_sum_norm_kernel<float><<<n, 256, smem, st>>>(static_cast<float*>(out), h, y, y_dtype, alpha, w, last_w, hidden, eps);
+  }
+  NVLLM_LAUNCH_CHECK("rms_sum_norm_kernel");
   return 0;
 }
 

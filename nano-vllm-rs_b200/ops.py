@@ -659,3 +659,103 @@ def embedding_stream(table, ids, scale, dtype):
     check(_ffi.lib().nvllm_embedding_stream(_p(h), _p(x), BF16 if dtype == torch.bfloat16 else F32, _p(table), _p(ids), n, hidden, table.shape[0],
                                             float(scale), _dt(table), _stream()))
     return h, x
+
+
+# ---- norm after the sum, weighted head norms before the rotation, kept first keys, per-head delta rule, gated linear attention
+
+
+def rms_sum_norm(h, y, alpha, w, eps, dtype, last_w=None):
+    """h = rms(alpha * h + y) * w in place (f32); returns h, or rms(h) * last_w, in `dtype`."""
+    n, hidden = h.shape
+    out = torch.empty((n, hidden), dtype=dtype, device=h.device)
+    check(_ffi.lib().nvllm_rms_sum_norm(_p(out), _p(h), _p(y), _dt(y), alpha, _p(w), _p(last_w), n, hidden, eps, _dt(out), _stream()))
+    return out
+
+
+def rope_table_scaled(max_pos, dims, base, device, scaling=None):
+    """[max_pos, dims / 2, 2] of (cos, sin); scaling: (factor, low, high, original) or None."""
+    tab = torch.empty((max_pos, dims // 2, 2), dtype=torch.float32, device=device)
+    f, lo, hi, orig = scaling if scaling is not None else (0.0, 1.0, 2.0, 1.0)
+    check(_ffi.lib().nvllm_rope_table_scaled(_p(tab), max_pos, dims, float(base), float(f), float(lo), float(hi), float(orig), _stream()))
+    return tab
+
+
+def attn_norm_rotary_store(proj, heads, kv_heads, dim, vdim, q_norm_w, k_norm_w, norm_eps, positions, table, rot_dims, halves, k_cache, v_cache,
+                           slots, dtype, v_first=None, v_lambda=None):
+    """Weighted RMS norm per query / key head, then the rotation; values stored, saved to v_first, or mixed with it (v_lambda)."""
+    n = proj.shape[0]
+    q = torch.empty((n, heads * dim), dtype=dtype, device=proj.device)
+    check(_ffi.lib().nvllm_attn_norm_rotary_store(_p(q), q.stride(0), _p(k_cache), _p(v_cache), k_cache.stride(0), v_cache.stride(0), _p(proj),
+                                                  proj.stride(0), _p(q_norm_w), _p(k_norm_w), float(norm_eps), _p(positions), _p(table), rot_dims,
+                                                  int(halves), table.shape[0] if table is not None else 1, _p(v_first),
+                                                  v_first.stride(0) if v_first is not None else 0, _p(v_lambda), _p(slots), n, heads, kv_heads,
+                                                  dim, vdim, _dt(q), _stream()))
+    return q
+
+
+def masked_attention(q, gate, k_cache, v_cache, tok_seq, positions, tables, block_size, heads, kv_heads, dim, vdim, scale, window=0, keep_first=0,
+                     sinks=None, gate_per_head=False, chunk=0, cu_tokens=None):
+    """window_attention whose first keep_first keys stay visible outside the window (or chunk)."""
+    n = q.shape[0]
+    out = torch.empty((n, heads * vdim), dtype=q.dtype, device=q.device)
+    check(_ffi.lib().nvllm_masked_attention(_p(out), out.stride(0), _p(q), q.stride(0), _p(gate), gate.stride(0) if gate is not None else 0,
+                                            int(gate_per_head), _p(k_cache), _p(v_cache), k_cache.stride(0), v_cache.stride(0), _p(tok_seq),
+                                            _p(positions), _p(tables), tables.shape[1] if tables is not None else 1, block_size, n, heads,
+                                            kv_heads, dim, vdim, scale, 0.0, 0.0, 1, window, keep_first, _p(sinks), chunk, None, None, 0, None, 0,
+                                            _p(cu_tokens), cu_tokens.shape[0] - 1 if cu_tokens is not None else 0, _dt(q), _stream()))
+    return out
+
+
+def head_delta_prepare(q, k, beta, decay, a_log, dt_bias, heads, groups, dk, q_scale, unit_eps=1e-6):
+    """delta_prepare with one decay per head: decay [n, heads], dt_bias [heads]."""
+    check(_ffi.lib().nvllm_head_delta_prepare(_p(q), q.stride(0), _p(k), k.stride(0), _p(beta), beta.stride(0), _p(decay), decay.stride(0), _p(a_log),
+                                              _p(dt_bias), q.shape[0], heads, groups, dk, q_scale, unit_eps, _stream()))
+
+
+def head_delta_recurrence(q, k, v, decay, beta, state, seq_slot, cu_tokens, positions, heads, groups, dk, dv):
+    """gated_delta_recurrence with one decay per head: decay [n, heads]."""
+    n = v.shape[0]
+    y = torch.empty((n, heads * dv), dtype=torch.float32, device=v.device)
+    check(_ffi.lib().nvllm_head_delta_recurrence(_p(y), y.stride(0), _p(q), q.stride(0), _p(k), k.stride(0), _p(v), v.stride(0), _p(decay),
+                                                 decay.stride(0), _p(beta), beta.stride(0), _p(state), _p(seq_slot), _p(cu_tokens),
+                                                 _p(positions), seq_slot.shape[0], heads, groups, dk, dv, _stream()))
+    return y
+
+
+def channel_recurrence(q, k, v, decay, q_scale, state, seq_slot, cu_tokens, positions, heads, groups, dk, dv):
+    """S <- diag(decay) S + k v^T, y = q_scale S^T q over the sequences of a step; decay [n, heads * dk]."""
+    n = v.shape[0]
+    y = torch.empty((n, heads * dv), dtype=torch.float32, device=v.device)
+    check(_ffi.lib().nvllm_channel_recurrence(_p(y), y.stride(0), _p(q), q.stride(0), _p(k), k.stride(0), _p(v), v.stride(0), _p(decay),
+                                              decay.stride(0), q_scale, _p(state), _p(seq_slot), _p(cu_tokens), _p(positions), seq_slot.shape[0],
+                                              heads, groups, dk, dv, _stream()))
+    return y
+
+
+def low_rank_decay(x, w2, bias, tau):
+    """sigmoid(x @ w2 + bias)^(1 / tau), f32; w2 [rank, channels]."""
+    n, (rank, ch) = x.shape[0], w2.shape
+    out = torch.empty((n, ch), dtype=torch.float32, device=x.device)
+    check(_ffi.lib().nvllm_low_rank_decay(_p(out), ch, _p(x), x.stride(0), _p(w2), _p(bias), n, rank, ch, tau, _stream()))
+    return out
+
+
+def gemm_glu(x, w_gate_up, limit):
+    """glu(x Wg^T, x Wu^T) with the clamped gate (limit > 0) or SiLU in the GEMM's epilogue; w_gate_up [2 inter, k]."""
+    _need(x, torch.bfloat16, "x"); _need(w_gate_up, torch.bfloat16, "w_gate_up")
+    M, K = x.shape
+    inter = w_gate_up.shape[0] // 2
+    out = torch.empty((M, inter), dtype=torch.bfloat16, device=x.device)
+    ws = torch.empty((M, 2 * inter), dtype=torch.bfloat16, device=x.device)
+    check(_ffi.lib().nvllm_gemm_glu_bf16(_p(out), _p(x), _p(w_gate_up), M, inter, K, x.stride(0), w_gate_up.stride(0), out.stride(0), limit, _p(ws),
+                                         ws.numel() * 2, _stream()))
+    return out
+
+
+def gemm_glu_grouped(x, w, tile_group, inter, groups, limit):
+    """gemm_glu over 128-row expert tiles; w [groups * 2 inter, k]."""
+    rows, K = x.shape
+    out = torch.empty((rows, inter), dtype=torch.bfloat16, device=x.device)
+    check(_ffi.lib().nvllm_gemm_glu_bf16_grouped(_p(out), _p(x), _p(w), rows, inter, K, groups, x.stride(0), w.stride(0), out.stride(0),
+                                                 _p(tile_group), limit, _stream()))
+    return out
