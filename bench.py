@@ -53,13 +53,15 @@ def parse():
     ap.add_argument("--warmup", type=int, default=4)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--model", default=None, help="override the workload model (qwen3-0.6b | qwen3-8b | qwen3-32b)")
-    ap.add_argument("--workload", default="decode", choices=["decode", "prefix", "kosazen", "talapel", "zudatar", "zasorax"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "prefix", "kosazen", "talapel", "zudatar", "zasorax", "kalesun"],
                     help="kosazen: prefill / decode throughput and a per-kernel roofline table of the Kosazen architecture "
                          "(latent attention + mixture of experts) beside Qwen3 models of equal layer sizes, random weights; "
                          "talapel: the same for the Talapel architecture (capped attention beside a state-space mixer, retention, "
                          "table-routed experts); zudatar: the same for the Zudatar architecture (windowed attention, latent "
                          "attention in a window, gated delta rule); zasorax: the same for the Zasorax architecture (post-norm blocks, "
-                         "chunked attention with a distance bias, rotated values, experts routed on logits)")
+                         "chunked attention with a distance bias, rotated values, experts routed on logits); kalesun: the Kalesun architecture "
+                         "(norm after the sum, windowed attention with kept first keys, gated delta rule, gated linear attention) beside "
+                         "Zudatar and Zasorax models of equal layer sizes")
     ap.add_argument("--seqs", type=int, default=None)
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-parity", action="store_true", help="skip the in-run parity checks (profiling runs)")
@@ -796,6 +798,32 @@ def zasorax_config(z):
             "layers": [kinds[i % 4] for i in range(z["layers"])]}
 
 
+# Kalesun: a gated-linear-attention layer, a windowed attention layer with experts, a delta-rule layer and a second attention
+# layer that mixes in the first one's values; the sizes (width, heads, window, feed-forward, experts) are those of the Zudatar
+# and Zasorax arms it is measured beside: its delta rule, window attention and dense layers have their like kernels in
+# the former, its experts and post-norm step in the latter.
+KALESUN_SIZES = {
+    "w2048": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=128, window=512, keep=4, rot_dims=64, d_heads=16, d_kv_heads=16, d_dim=128, d_vdim=128,
+                  taps=4, l_heads=16, l_dim=128, l_vdim=128, low_rank=16, dense_ff=8192, ff=1024, experts=32, top=4, layers=4, vocab=32768),
+    "w4096": dict(width=4096, heads=32, kv_heads=8, dim=128, vdim=128, window=512, keep=4, rot_dims=64, d_heads=32, d_kv_heads=32, d_dim=128, d_vdim=128,
+                  taps=4, l_heads=32, l_dim=128, l_vdim=128, low_rank=16, dense_ff=12288, ff=1536, experts=32, top=4, layers=4, vocab=32768),
+}
+
+
+def kalesun_config(z):
+    dense = {"kind": "dense", "ff": z["dense_ff"], "limit": 7.0}
+    moe = {"kind": "moe", "expert": {"ff": z["ff"], "limit": 7.0}, "router": {"experts": z["experts"], "top": z["top"]}}
+    att = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["vdim"], "scale": z["dim"] ** -0.5, "v_mix": True,
+           "mask": {"size": z["window"], "keep_first": z["keep"]},
+           "rot": {"base": 500000.0, "dims": z["rot_dims"], "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    dlt = {"heads": z["d_heads"], "kv_heads": z["d_kv_heads"], "dim": z["d_dim"], "vdim": z["d_vdim"], "conv": z["taps"]}
+    gla = {"heads": z["l_heads"], "dim": z["l_dim"], "vdim": z["l_vdim"], "tau": 16.0, "low_rank": z["low_rank"]}
+    kinds = [{"type": "gla", "mixer": gla, "mlp": dense}, {"type": "attention", "mixer": att, "mlp": moe},
+             {"type": "delta", "mixer": dlt, "mlp": dense}, {"type": "attention", "mixer": att, "mlp": moe}]
+    return {"architecture": "Kalesun", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5}, "postln_alpha": 1.5,
+            "layers": [kinds[i % 4] for i in range(z["layers"])]}
+
+
 def kernel_rooflines(z, arch, n_tok, ctx, decode, hbm, tf):
     """Algorithmic work of the named launches of ONE layer at n_tok tokens (context ctx per sequence): {name: (flop, bytes)}."""
     W, H, L = z["width"], z["heads"], ctx
@@ -858,6 +886,42 @@ def kernel_rooflines(z, arch, n_tok, ctx, decode, hbm, tf):
         out["moe_combine"] = (0, n_tok * (z["top"] + 1) * W * 2)
         out["rms_residual_norm"] = (0, n_tok * W * (4 + 4 + 2 + 2))
         return {k: max(f / (tf * 1e12), b / (hbm * 1e9)) * 1e6 for k, (f, b) in out.items()}
+    if arch == "kalesun":
+        D, V, G, w = z["dim"], z["vdim"], z["kv_heads"], z["window"]
+        dH, dG, dD, dV = z["d_heads"], z["d_kv_heads"], z["d_dim"], z["d_vdim"]
+        lH, lD, lV, lr = z["l_heads"], z["l_dim"], z["l_vdim"], z["low_rank"]
+        seqs = n_tok if decode else max(1, n_tok // L)
+        # (query, key) pairs per head: the window and, where it no longer reaches them, the kept first keys
+        see = min(L, w + z["keep"])
+        wpairs = n_tok * see if decode else seqs * sum(min(p + 1, w + z["keep"]) for p in range(L))
+        gemm = lambda n, k: (2 * n_tok * n * k, 2 * n * k + n_tok * (2 * k + 4 * n))
+        qkv = H * D + G * D + G * V
+        out["attention q k v g projection"] = gemm(qkv + H, W)
+        out["attn_norm_rotary_store"] = (0, n_tok * (qkv * 6 + G * V * 4))
+        out["masked_attention"] = (2 * wpairs * H * (D + V), (n_tok * see if decode else n_tok) * G * (D + V) * 2 + n_tok * H * (D + V) * 2)
+        ch = 2 * dG * dD + dH * dV
+        out["delta q k v g b a projection"] = gemm(ch + dH * dV + 2 * dH, W)
+        out["causal_conv"] = (2 * n_tok * ch * z["taps"], n_tok * ch * 8)
+        out["head_delta_prepare"] = (0, n_tok * 2 * dG * dD * 8)
+        # per state element and token 8 flop (decay, two read-outs, the write) of the delta rule and 6 of gated linear attention
+        # (decay, write, read-out); the state is read and written once per portion
+        out["head_delta_recurrence"] = (8 * n_tok * dH * dD * dV, n_tok * (2 * dG * dD + 2 * dH * dV) * 4 + seqs * dH * dD * dV * 8)
+        out["gla q k v g a1 projection"] = gemm(2 * lH * lD + 2 * lH * lV + lr, W)
+        out["low_rank_decay"] = (2 * n_tok * lr * lH * lD, n_tok * (lr + lH * lD) * 4)
+        out["channel_recurrence"] = (6 * n_tok * lH * lD * lV, n_tok * (3 * lH * lD + 2 * lH * lV) * 4 + seqs * lH * lD * lV * 8)
+        out["gated_group_norm"] = (0, n_tok * (dH * dV + lH * lV) // 2 * 10)
+        out["mixer output projection"] = gemm(W, H * V)
+        out["gate / up projection + clamped gate"] = (2 * n_tok * W * 2 * z["dense_ff"], 2 * W * 2 * z["dense_ff"] + n_tok * 2 * (W + z["dense_ff"]))
+        out["down projection"] = (2 * n_tok * W * z["dense_ff"], 2 * W * z["dense_ff"] + n_tok * 2 * (W + z["dense_ff"]))
+        used = min(z["experts"], n_tok * z["top"])
+        out["expert gate / up + clamped gate grouped GEMM"] = (2 * n_tok * z["top"] * W * 2 * z["ff"], 2 * used * 2 * z["ff"] * W)
+        out["expert down grouped GEMM"] = (2 * n_tok * z["top"] * W * z["ff"], 2 * used * z["ff"] * W)
+        out["expert row gather"] = (0, n_tok * z["top"] * W * 4)
+        out["moe_combine"] = (0, n_tok * (z["top"] + 1) * W * 2)
+        out["rms_sum_norm"] = out["rms_sum_norm (+ final norm)"] = (0, n_tok * W * (4 + 4 + 2 + 2))
+        f32_tf = 148 * 128 * 2 * 1.965e9 / 1e12   # everything that enters a recurrence is f32 by definition of the design
+        f32_names = ("head_delta_recurrence", "channel_recurrence", "low_rank_decay", "causal_conv")
+        return {k: max(f / ((f32_tf if k in f32_names else tf) * 1e12), b / (hbm * 1e9)) * 1e6 for k, (f, b) in out.items()}
     if arch == "zudatar":
         D, V, G, R, QR, w = z["dim"], z["vdim"], z["kv_heads"], z["kv_rank"], z["q_rank"], z["window"]
         dH, dG, dD, dV, lr = z["d_heads"], z["d_kv_heads"], z["d_dim"], z["d_vdim"], z["low_rank"]
@@ -886,6 +950,9 @@ def kernel_rooflines(z, arch, n_tok, ctx, decode, hbm, tf):
         out["causal_conv"] = (2 * n_tok * ch * z["taps"], n_tok * ch * 8)
         # 8 flop per state element and token (decay, two read-outs, the write); the state is read and written once per portion
         out["gated_delta_recurrence"] = (8 * n_tok * dH * dD * dV, n_tok * (2 * dG * dD + dH * dD + 2 * dH * dV) * 4 + seqs * dH * dD * dV * 8)
+        out["delta_prepare"] = (0, n_tok * (2 * dG * dD + dH * dD) * 8)
+        out["gated_group_norm"] = (0, n_tok * dH * dV * 10)
+        out["attn_rope_norm_store"] = (0, n_tok * (H * D + 2 * G * D) * 6)
         out["gate_up projection"] = out["gate_up projection + SiLU gate"] = gemm(2 * z["dense_ff"], W)
         out["down projection"] = gemm(W, z["dense_ff"])
         out["rms_residual_norm"] = (0, n_tok * W * (4 + 4 + 4 + 2))
@@ -913,16 +980,17 @@ def kernel_rooflines(z, arch, n_tok, ctx, decode, hbm, tf):
     return {k: max(f / (tf * 1e12), b / (hbm * 1e9)) * 1e6 for k, (f, b) in out.items()}   # roofline microseconds
 
 
-def run_arch_compare(args, new_arch="kosazen"):
+def run_arch_compare(args, new_arch="kosazen", beside=("qwen3",)):
     import torch
     from nano_vllm_rs_b200 import engine as E
     hbm, _ = peaks()
     tf, _ = tensor_peak()
     n_prompts, plen, dec_b = 8, 1024, args.seqs or 64
     rng = __import__("numpy").random.default_rng(0)
-    result = {"workload": f"{new_arch}-vs-qwen3", "data": "synthetic", "dtype": "bf16", "prefill": f"{n_prompts} x {plen} tokens per step",
+    result = {"workload": f"{new_arch}-vs-{'-'.join(beside)}", "data": "synthetic", "dtype": "bf16", "prefill": f"{n_prompts} x {plen} tokens per step",
               "decode": f"{dec_b} sequences at context {plen}+", "peaks": {"hbm_gbs": hbm, "bf16_tflops": tf}, "sizes": {}}
-    sizes = {"kosazen": ARCH_SIZES, "talapel": TALAPEL_SIZES, "zudatar": ZUDATAR_SIZES, "zasorax": ZASORAX_SIZES}[new_arch]
+    all_sizes = {"kosazen": ARCH_SIZES, "talapel": TALAPEL_SIZES, "zudatar": ZUDATAR_SIZES, "zasorax": ZASORAX_SIZES, "kalesun": KALESUN_SIZES}
+    sizes = all_sizes[new_arch]
     only = os.environ.get("BENCH_ARCH_SIZES")          # e.g. "w2048": a subset of the sizes
     for name, z in sizes.items():
         if only and name not in only.split(","):
@@ -937,9 +1005,11 @@ def run_arch_compare(args, new_arch="kosazen"):
             z = dict(z, shared_ff=0)
             mlp_q = (2 * z["dense_ff"] + 3 * 3 * z["top"] * z["ff"]) // 12 // 64 * 64
         else:
-            mlp_q = z["top"] * z["ff"] + z["shared_ff"]
+            mlp_q = z["top"] * z["ff"] + z.get("shared_ff", 0)
         result["sizes"][name] = {}
-        for arch in (new_arch, "qwen3"):
+        for arch in (new_arch,) + tuple(beside):
+            if arch != new_arch and arch != "qwen3":
+                z = all_sizes[arch][name]
             progress(f"{name} {arch}: building the engine (random weights)")
             blocks = dec_b * (plen + 256) // 256 + 8
             common = dict(kvcache_block_size=256, num_kvcache_blocks=blocks, max_num_seqs=dec_b,
@@ -952,6 +1022,8 @@ def run_arch_compare(args, new_arch="kosazen"):
                 cfg = E.Config(model_config=zudatar_config(z), **common)
             elif arch == "zasorax":
                 cfg = E.Config(model_config=zasorax_config(z), **common)
+            elif arch == "kalesun":
+                cfg = E.Config(model_config=kalesun_config(z), **common)
             else:
                 cfg = E.Config("qwen3-0.6b", vocab_size=z["vocab"], hidden_size=z["width"], num_hidden_layers=z["layers"],
                                intermediate_size=mlp_q, num_attention_heads=z["heads"],
@@ -1056,6 +1128,10 @@ def main():
     torch.cuda.set_device(local)
     lib = E.lib()
     assert lib.nvllm_device_ok() == 1, "no sm_100 device: the product path has no fallback"
+    if args.workload == "kalesun":
+        assert world == 1, "--workload kalesun is a one-GPU comparison"
+        print(json.dumps(run_arch_compare(args, "kalesun", ("zudatar", "zasorax"))), flush=True)
+        return 0
     if args.workload == "zasorax":
         assert world == 1, "--workload zasorax is a one-GPU comparison"
         print(json.dumps(run_arch_compare(args, "zasorax")), flush=True)

@@ -153,9 +153,7 @@ __device__ __forceinline__ uint32_t pack_bf16x2(float lo, float hi) {
   bf162 v = __floats2bfloat162_rn(lo, hi);  // .x = lo (low 16 bits)
   return *reinterpret_cast<uint32_t*>(&v);
 }
-// One pair of a gated feed-forward's activations from bf16 pre-activations (gb: two gates, ub: two ups).
-//   limit <= 0: silu(g) u, silu rounded to bf16 (the rounding points of a separate activation kernel)
-//   limit > 0:  g' sigmoid(1.702 g') (u' + 1) with g' = min(g, limit) and u' = u clamped to [-limit, limit]
+// The clamped gate of a feed-forward: g' sigmoid(1.702 g') (u' + 1) with g' = min(g, limit), u' = u clamped to [-limit, limit].
 __device__ __forceinline__ float bf16_lo(uint32_t v);
 __device__ __forceinline__ float bf16_hi(uint32_t v);
 __device__ __forceinline__ float glu_clamped(float g, float u, float limit) {
@@ -163,9 +161,18 @@ __device__ __forceinline__ float glu_clamped(float g, float u, float limit) {
   u = fminf(fmaxf(u, -limit), limit);
   return g * (1.0f / (1.0f + expf(-1.702f * g))) * (u + 1.0f);
 }
+// The same where a bf16 result follows (GEMM epilogues): exponential and division in their fast forms.
+__device__ __forceinline__ float glu_clamped_fast(float g, float u, float limit) {
+  g = fminf(g, limit);
+  return __fdividef(g, 1.0f + __expf(-1.702f * g)) * (fminf(fmaxf(u, -limit), limit) + 1.0f);
+}
+// One pair of a gated feed-forward's activations from bf16 pre-activations (gb: two gates, ub: two ups) in a GEMM epilogue.
+// GATE 1: silu(g) u, silu rounded to bf16 (the rounding points of a separate activation kernel); GATE 2: the clamped gate.
+enum { kGateNone = 0, kGateSilu = 1, kGateClamped = 2 };
+template <int GATE>
 __device__ __forceinline__ float2 gated_pair(uint32_t gb, uint32_t ub, float limit) {
   const float g0 = bf16_lo(gb), g1 = bf16_hi(gb);
-  if (limit > 0.f) return make_float2(glu_clamped(g0, bf16_lo(ub), limit), glu_clamped(g1, bf16_hi(ub), limit));
+  if (GATE == kGateClamped) return make_float2(glu_clamped_fast(g0, bf16_lo(ub), limit), glu_clamped_fast(g1, bf16_hi(ub), limit));
   const uint32_t sb = pack_bf16x2(g0 / (1.0f + expf(-g0)), g1 / (1.0f + expf(-g1)));
   return make_float2(bf16_lo(sb) * bf16_lo(ub), bf16_hi(sb) * bf16_hi(ub));
 }

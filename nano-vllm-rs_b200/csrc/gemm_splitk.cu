@@ -72,8 +72,8 @@ __device__ __forceinline__ void st_smem_f32(uint32_t addr, float v) {
 }
 
 // One cluster of SK CTAs per (m_tile, n_tile); cluster rank r accumulates k-blocks [r * kb_per, (r + 1) * kb_per).
-// SILU: w = [gate (N rows) | up (N rows)], the B tile is BN/2 gate rows + the matching BN/2 up rows, y[:, BN/2 per tile].
-template <int BN, int SK, bool SILU>
+// GATE: w = [gate (N rows) | up (N rows)], the B tile is BN/2 gate rows + the matching BN/2 up rows, y[:, BN/2 per tile].
+template <int BN, int SK, int GATE>
 __global__ void __launch_bounds__(256, 1)
 gemm_splitk_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_constant__ CUtensorMap tmap_w,
                    bf16* __restrict__ y, int M, int N, int K, int64_t ldy, int num_m_tiles, int STAGES, const RowPush ps, float glu_limit) {
@@ -117,7 +117,7 @@ gemm_splitk_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_cons
   if (warp == 0 && lane == 0) {
     // ===== TMA producer: weights first (independent of the predecessor kernel), x after the dependency wait =====
     auto load_w = [&](int stage, int kb) {
-      if constexpr (SILU) {
+      if constexpr (GATE != kGateNone) {
         tma_load_2d(sB + stage * C::kBBytes, &tmap_w, full_bar(stage), kb * C::BK, n_tile * (BN / 2));
         tma_load_2d(sB + stage * C::kBBytes + (BN / 2) * 128, &tmap_w, full_bar(stage), kb * C::BK, N + n_tile * (BN / 2));
       } else {
@@ -195,7 +195,7 @@ gemm_splitk_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_cons
     uint32_t peer[SK];
 #pragma unroll
     for (int r = 0; r < SK; ++r) peer[r] = dsmem_addr(smem_base + row_in * 4, static_cast<uint32_t>(r));
-    if constexpr (SILU) {
+    if constexpr (GATE != kGateNone) {
       constexpr int CW = BN / (2 * SK);  // output columns of this CTA
       static_assert(CW >= 8 && CW % 8 == 0, "slice must be whole 16-byte vectors");
       bf16* dst = y + row * ldy + n_tile * (BN / 2) + rank * CW;
@@ -223,7 +223,7 @@ gemm_splitk_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_cons
         for (int e = 0; e < 8; e += 2) {  // rounding points of the unfused path: bf16 gate_up, bf16 silu(gate), bf16 product
           const uint32_t gb = pack_bf16x2(g[e], g[e + 1]);
           const uint32_t ub = pack_bf16x2(u[e], u[e + 1]);
-          const float2 p = gated_pair(gb, ub, glu_limit);
+          const float2 p = gated_pair<GATE>(gb, ub, glu_limit);
           o[e / 2] = pack_bf16x2(p.x, p.y);
         }
         if (row < M) *reinterpret_cast<uint4*>(dst + j) = make_uint4(o[0], o[1], o[2], o[3]);
@@ -300,11 +300,11 @@ int splitk_stages(int kb_per) {
   return want < kb_per ? want : (kb_per < 1 ? 1 : kb_per);
 }
 
-template <int BN, int SK, bool SILU>
+template <int BN, int SK, int GATE>
 int launch_splitk(const CUtensorMap& tx, const CUtensorMap& tw, void* y, int M, int N, int K, int64_t ldy, int tiles,
                   int num_m_tiles, cudaStream_t st, const RowPush& ps, float glu_limit = 0.f) {
   using C = SkCfg<BN>;
-  auto kern = gemm_splitk_kernel<BN, SK, SILU>;
+  auto kern = gemm_splitk_kernel<BN, SK, GATE>;
   NVLLM_SMEM_ATTR_ONCE(kern, C::smem_bytes(C::kMaxStages));
   const int stages = splitk_stages<BN>((K / C::BK) / SK);
   cudaLaunchConfig_t cfg{};
@@ -381,16 +381,17 @@ namespace nvllm {
 #endif
 
 int gemm_splitk_dispatch(void* y, const void* x, const void* w, int m, int n, int k, int64_t ldx, int64_t ldw, int64_t ldy,
-                         bool silu, int bn, int sk, cudaStream_t st, const RowPush& ps, float glu_limit) {
+                         bool gated, int bn, int sk, cudaStream_t st, const RowPush& ps, float glu_limit) {
   CUtensorMap tx, tw;
-  const int n_acc = silu ? 2 * n : n;
+  const int n_acc = gated ? 2 * n : n;
   if (int rc = make_tmap_bf16_2d(&tx, x, m, k, ldx, 128)) return rc;
-  if (int rc = make_tmap_bf16_2d(&tw, w, n_acc, k, ldw, silu ? bn / 2 : bn)) return rc;
+  if (int rc = make_tmap_bf16_2d(&tw, w, n_acc, k, ldw, gated ? bn / 2 : bn)) return rc;
   const int mt = (m + 127) / 128, tiles = mt * (n_acc / bn);
 #define NVLLM_SK(BNV, SKV)                                                                                   \
   if (bn == BNV && sk == SKV)                                                                                \
-    return silu ? launch_splitk<BNV, SKV, true>(tx, tw, y, m, n, k, ldy, tiles, mt, st, RowPush{}, glu_limit)                      \
-                : launch_splitk<BNV, SKV, false>(tx, tw, y, m, n, k, ldy, tiles, mt, st, ps)
+    return !gated           ? launch_splitk<BNV, SKV, kGateNone>(tx, tw, y, m, n, k, ldy, tiles, mt, st, ps)                        \
+           : glu_limit > 0.f ? launch_splitk<BNV, SKV, kGateClamped>(tx, tw, y, m, n, k, ldy, tiles, mt, st, RowPush{}, glu_limit) \
+                             : launch_splitk<BNV, SKV, kGateSilu>(tx, tw, y, m, n, k, ldy, tiles, mt, st, RowPush{})
   NVLLM_SK(256, 8); NVLLM_SK(256, 4); NVLLM_SK(256, 2);
   NVLLM_SK(128, 8); NVLLM_SK(128, 4); NVLLM_SK(128, 2);
   NVLLM_SK(64, 4); NVLLM_SK(64, 2);

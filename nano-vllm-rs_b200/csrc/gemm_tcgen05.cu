@@ -73,7 +73,7 @@ __device__ __forceinline__ void store_row32<float>(float* dst, const uint32_t (&
   }
 }
 
-// SILU == true: w = [gate (N rows) | up (N rows)]; the B tile is staged as BN/2 gate rows + the matching BN/2 up rows and
+// GATE != kGateNone: w = [gate (N rows) | up (N rows)]; the B tile is staged as BN/2 gate rows + the matching BN/2 up rows and
 // the epilogue writes y[:, n_tile*BN/2 + c] = silu(gate) * up, or with glu_limit > 0 the clamped gate of gated_pair (see gemm_tcgen05_2cta.cu for the CTA-pair variant).
 // Optional qkv epilogue (ROPE mode, BN == 128 == head_dim): each output tile is one head of the packed [q | k | v] row,
 // and each epilogue thread owns that head for one token.  It applies what Qwen3Attention::forward does between qkv_proj
@@ -96,7 +96,7 @@ struct RopeEpi {
 // CN > 1: clusters of CN CTAs along N work on the same 128-row x tile.  Each CTA loads 128/CN rows of it and MULTICASTS
 // them into all CN shared memories (L2 -> SM traffic for x drops by CN: the bound for small-N, long-K shards such as the
 // TP=8 qkv / o / down projections); a stage is released only when all CN CTAs' MMAs have retired (multicast commit).
-template <int BN, typename OutT, bool SILU, int CN, bool ROPE = false>
+template <int BN, typename OutT, int GATE, int CN, bool ROPE = false>
 __global__ void __launch_bounds__(256, 1)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_constant__ CUtensorMap tmap_w,
                     OutT* __restrict__ y, int M, int N, int K, int64_t ldy, int num_m_tiles, int num_tiles,
@@ -152,7 +152,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_con
     // The weights do not depend on the previous kernel: the first ring of w tiles is requested BEFORE the
     // programmatic-dependency wait, so their HBM latency hides behind the predecessor's tail; x follows after it.
     auto load_w = [&](int stage, int kb, int n_tile, int goff = 0) {
-      if constexpr (SILU) {
+      if constexpr (GATE != kGateNone) {
         tma_load_2d(sB + stage * C::kBBytes, &tmap_w, full_bar(stage), kb * C::BK, goff + n_tile * (BN / 2));
         tma_load_2d(sB + stage * C::kBBytes + (BN / 2) * 128, &tmap_w, full_bar(stage), kb * C::BK, goff + N + n_tile * (BN / 2));
       } else {
@@ -298,7 +298,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_con
             }
           }
         }
-      } else if constexpr (SILU) {
+      } else if constexpr (GATE != kGateNone) {
 #pragma unroll 1
         for (int c = 0; c < BN / 64; ++c) {
           uint32_t g[32], u[32];
@@ -309,7 +309,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_con
           for (int e = 0; e < 32; e += 2) {  // rounding points of the unfused path: bf16 gate_up, bf16 silu(gate)
             const uint32_t gb = pack_bf16x2(__uint_as_float(g[e]), __uint_as_float(g[e + 1]));
             const uint32_t ub = pack_bf16x2(__uint_as_float(u[e]), __uint_as_float(u[e + 1]));
-            const float2 p = gated_pair(gb, ub, glu_limit);
+            const float2 p = gated_pair<GATE>(gb, ub, glu_limit);
             g[e] = __float_as_uint(p.x);
             g[e + 1] = __float_as_uint(p.y);
           }
@@ -347,15 +347,15 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_con
   }
 }
 
-template <int BN, typename OutT, bool SILU = false, int CN = 1, bool ROPE = false>
+template <int BN, typename OutT, int GATE = kGateNone, int CN = 1, bool ROPE = false>
 static int launch_gemm(const CUtensorMap& tx, const CUtensorMap& tw, void* y, int M, int N, int K, int64_t ldy,
                        cudaStream_t st, const RopeEpi& re = RopeEpi{}, const RowPush& ps = RowPush{},
                        const int32_t* tile_group = nullptr, int group_rows = 0, float glu_limit = 0.f) {
   using C = GemmCfg<BN>;
-  auto kern = gemm_tcgen05_kernel<BN, OutT, SILU, CN, ROPE>;
+  auto kern = gemm_tcgen05_kernel<BN, OutT, GATE, CN, ROPE>;
   NVLLM_SMEM_ATTR_ONCE(kern, C::kSmemBytes);
   const int num_m_tiles = (M + C::BM - 1) / C::BM;
-  const int num_n_tiles = SILU ? (N + BN / 2 - 1) / (BN / 2) : (N + BN - 1) / BN;
+  const int num_n_tiles = GATE != kGateNone ? (N + BN / 2 - 1) / (BN / 2) : (N + BN - 1) / BN;
   const int num_tiles = num_m_tiles * (num_n_tiles / CN);  // cluster tiles (the caller guarantees num_n_tiles % CN == 0)
   const int max_clusters = sm_count() / CN;
   const int clusters = num_tiles < max_clusters ? num_tiles : max_clusters;
@@ -388,6 +388,13 @@ static int launch_gemm(const CUtensorMap& tx, const CUtensorMap& tw, void* y, in
                                   static_cast<int>(C::kStages), ps, tile_group, group_rows, glu_limit));
   }
   return 0;
+}
+
+template <int BN>
+static int launch_gated(const CUtensorMap& tx, const CUtensorMap& tw, void* y, int m, int inter, int k, int64_t ldy, float limit, cudaStream_t st,
+                        const int32_t* tile_group = nullptr) {
+  if (limit > 0.f) return launch_gemm<BN, bf16, kGateClamped>(tx, tw, y, m, inter, k, ldy, st, RopeEpi{}, RowPush{}, tile_group, 2 * inter, limit);
+  return launch_gemm<BN, bf16, kGateSilu>(tx, tw, y, m, inter, k, ldy, st, RopeEpi{}, RowPush{}, tile_group, 2 * inter);
 }
 
 static int pick_bn(int M, int N) {
@@ -486,8 +493,8 @@ int gemm_bf16_impl(void* y, const void* x, const void* w, int32_t m, int32_t n, 
   if (!push && use_mcast() && bn <= 64 && n % (4 * bn) == 0 && k >= 2048 && out_dtype == NVLLM_BF16) {
     if (int rc = make_tmap_bf16_2d(&tx, x, m, k, ldx, 32)) return rc;
     if (int rc = make_tmap_bf16_2d(&tw, w, n, k, ldw, bn)) return rc;
-    return bn == 64 ? launch_gemm<64, bf16, false, 4>(tx, tw, y, m, n, k, ldy, st)
-                    : launch_gemm<32, bf16, false, 4>(tx, tw, y, m, n, k, ldy, st);
+    return bn == 64 ? launch_gemm<64, bf16, kGateNone, 4>(tx, tw, y, m, n, k, ldy, st)
+                    : launch_gemm<32, bf16, kGateNone, 4>(tx, tw, y, m, n, k, ldy, st);
   }
   if (int rc = make_tmap_bf16_2d(&tx, x, m, k, ldx, 128)) return rc;
   if (int rc = make_tmap_bf16_2d(&tw, w, n, k, ldw, bn)) return rc;
@@ -555,8 +562,8 @@ extern "C" int nvllm_gemm_glu_bf16_grouped(void* y, const void* x, const void* w
   CUtensorMap tx, tw;
   if (int rc = make_tmap_bf16_2d(&tx, x, max_rows, k, ldx, 128)) return rc;
   if (int rc = make_tmap_bf16_2d(&tw, w, static_cast<int64_t>(groups) * 2 * inter, k, ldw, bn / 2)) return rc;
-  if (bn == 256) return launch_gemm<256, bf16, true>(tx, tw, y, max_rows, inter, k, ldy, st, RopeEpi{}, RowPush{}, tile_group, 2 * inter, limit);
-  return launch_gemm<128, bf16, true>(tx, tw, y, max_rows, inter, k, ldy, st, RopeEpi{}, RowPush{}, tile_group, 2 * inter, limit);
+  if (bn == 256) return launch_gated<256>(tx, tw, y, max_rows, inter, k, ldy, limit, st, tile_group);
+  return launch_gated<128>(tx, tw, y, max_rows, inter, k, ldy, limit, st, tile_group);
 }
 
 // MergedColumnParallelLinear::forward + SiluAndMul::forward in one call (linear.rs:437-439 + activation.rs:46-63).
@@ -592,10 +599,10 @@ extern "C" int nvllm_gemm_glu_bf16(void* out, const void* x, const void* w_gate_
     if (int rc = make_tmap_bf16_2d(&tx, x, m, k, ldx, 128)) return rc;
     if (int rc = make_tmap_bf16_2d(&tw, w_gate_up, 2 * static_cast<int64_t>(inter), k, ldw, bn / 2)) return rc;
     switch (bn) {
-      case 256: return launch_gemm<256, bf16, true>(tx, tw, out, m, inter, k, ldout, st, RopeEpi{}, RowPush{}, nullptr, 0, limit);
-      case 192: return launch_gemm<192, bf16, true>(tx, tw, out, m, inter, k, ldout, st, RopeEpi{}, RowPush{}, nullptr, 0, limit);
-      case 128: return launch_gemm<128, bf16, true>(tx, tw, out, m, inter, k, ldout, st, RopeEpi{}, RowPush{}, nullptr, 0, limit);
-      default: return launch_gemm<64, bf16, true>(tx, tw, out, m, inter, k, ldout, st, RopeEpi{}, RowPush{}, nullptr, 0, limit);
+      case 256: return launch_gated<256>(tx, tw, out, m, inter, k, ldout, limit, st);
+      case 192: return launch_gated<192>(tx, tw, out, m, inter, k, ldout, limit, st);
+      case 128: return launch_gated<128>(tx, tw, out, m, inter, k, ldout, limit, st);
+      default: return launch_gated<64>(tx, tw, out, m, inter, k, ldout, limit, st);
     }
   }
   // odd intermediate sizes: plain GEMM into the workspace, then the SiLU*mul kernel
@@ -640,5 +647,5 @@ extern "C" int nvllm_gemm_qkv_rope_store(void* qkv, const void* x, const void* w
   CUtensorMap tx, tw;
   if (int rc = make_tmap_bf16_2d(&tx, x, m, k, ldx, 128)) return rc;
   if (int rc = make_tmap_bf16_2d(&tw, w_qkv, n, k, ldw, 128)) return rc;
-  return launch_gemm<128, bf16, false, 1, true>(tx, tw, qkv, m, n, k, n, static_cast<cudaStream_t>(stream), re);
+  return launch_gemm<128, bf16, kGateNone, 1, true>(tx, tw, qkv, m, n, k, n, static_cast<cudaStream_t>(stream), re);
 }

@@ -46,11 +46,11 @@ __device__ __forceinline__ void store_row32_2(OutT* dst, const uint32_t (&r)[32]
   }
 }
 
-// SILU == true: w is the packed [gate (N rows) | up (N rows)] matrix of MergedColumnParallelLinear (linear.rs:421-433);
+// GATE != kGateNone: w is the packed [gate (N rows) | up (N rows)] matrix of MergedColumnParallelLinear (linear.rs:421-433);
 // the leader CTA stages BN/2 gate rows, its peer the matching BN/2 up rows, so accumulator columns [0, BN/2) are gate and
 // [BN/2, BN) are up for the same BN/2 output features, and the epilogue writes y[:, n_tile*BN/2 + c] = silu(gate)*up
 // (SiluAndMul::forward, activation.rs:46-63; glu_limit > 0: the clamped gate of gated_pair) without the [M, 2N] intermediate ever reaching HBM.  N = output features.
-template <int BN, typename OutT, bool SILU>
+template <int BN, typename OutT, int GATE>
 __global__ void __launch_bounds__(256, 1)
 gemm_tcgen05_2cta_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_constant__ CUtensorMap tmap_w,
                          OutT* __restrict__ y, int M, int N, int K, int64_t ldy, int num_m_tiles, int num_tiles, float glu_limit) {
@@ -108,7 +108,7 @@ gemm_tcgen05_2cta_kernel(const __grid_constant__ CUtensorMap tmap_x, const __gri
         if (leader) mbar_expect_tx(full_bar(stage), 2 * C::kStageBytes);
         tma_load_2d_cg2(sA + stage * C::kABytes, &tmap_x, full_bar(stage), kb * C::BK, m_tile * C::BM + rank * C::BM_CTA);
         tma_load_2d_cg2(sB + stage * C::kBBytes, &tmap_w, full_bar(stage), kb * C::BK,
-                        SILU ? static_cast<int>(rank) * N + n_tile * (BN / 2) : n_tile * BN + static_cast<int>(rank) * (BN / 2));
+                        GATE != kGateNone ? static_cast<int>(rank) * N + n_tile * (BN / 2) : n_tile * BN + static_cast<int>(rank) * (BN / 2));
         if (++stage == STAGES) { stage = 0; phase ^= 1; }
       }
     }
@@ -150,7 +150,7 @@ gemm_tcgen05_2cta_kernel(const __grid_constant__ CUtensorMap tmap_x, const __gri
       tc_fence_after();
       const int row = m_tile * C::BM + rank * C::BM_CTA + q * 32 + lane;
       const uint32_t taddr = tmem_base + (static_cast<uint32_t>(q * 32) << 16) + acc * BN;
-      if constexpr (SILU) {
+      if constexpr (GATE != kGateNone) {
 #pragma unroll 1
         for (int c = 0; c < BN / 64; ++c) {
           uint32_t g[32], u[32];
@@ -162,7 +162,7 @@ gemm_tcgen05_2cta_kernel(const __grid_constant__ CUtensorMap tmap_x, const __gri
             // same rounding points as the unfused path: gate_up is a bf16 tensor, silu(gate) is a bf16 tensor
             const uint32_t gb = pack_bf16x2(__uint_as_float(g[e]), __uint_as_float(g[e + 1]));
             const uint32_t ub = pack_bf16x2(__uint_as_float(u[e]), __uint_as_float(u[e + 1]));
-            const float2 p = gated_pair(gb, ub, glu_limit);
+            const float2 p = gated_pair<GATE>(gb, ub, glu_limit);
             g[e] = __float_as_uint(p.x);
             g[e + 1] = __float_as_uint(p.y);
           }
@@ -193,14 +193,14 @@ gemm_tcgen05_2cta_kernel(const __grid_constant__ CUtensorMap tmap_x, const __gri
   }
 }
 
-template <int BN, typename OutT, bool SILU = false>
+template <int BN, typename OutT, int GATE = kGateNone>
 static int launch_gemm2(const CUtensorMap& tx, const CUtensorMap& tw, void* y, int M, int N, int K, int64_t ldy,
                         cudaStream_t st, float glu_limit = 0.f) {
   using C = Gemm2Cfg<BN>;
-  auto kern = gemm_tcgen05_2cta_kernel<BN, OutT, SILU>;
+  auto kern = gemm_tcgen05_2cta_kernel<BN, OutT, GATE>;
   NVLLM_SMEM_ATTR_ONCE(kern, C::kSmemBytes);
   const int num_m_tiles = (M + C::BM - 1) / C::BM;
-  const int num_n_tiles = SILU ? (N + BN / 2 - 1) / (BN / 2) : (N + BN - 1) / BN;
+  const int num_n_tiles = GATE != kGateNone ? (N + BN / 2 - 1) / (BN / 2) : (N + BN - 1) / BN;
   const int num_tiles = num_m_tiles * num_n_tiles;
   const int max_clusters = sm_count() / 2;
   const int clusters = num_tiles < max_clusters ? num_tiles : max_clusters;
@@ -270,11 +270,17 @@ int gemm_silu_2cta_dispatch(void* y, const void* x, const void* w, int m, int in
   CUtensorMap tx, tw;
   if (int rc = make_tmap_bf16_2d(&tx, x, m, k, ldx, 128)) return rc;
   if (int rc = make_tmap_bf16_2d(&tw, w, 2 * static_cast<int64_t>(inter), k, ldw, bn / 2)) return rc;
+#define NVLLM_G2G(BNV)                                                                                                    \
+  case BNV:                                                                                                               \
+    return glu_limit > 0.f ? launch_gemm2<BNV, bf16, kGateClamped>(tx, tw, y, m, inter, k, ldy, st, glu_limit)            \
+                           : launch_gemm2<BNV, bf16, kGateSilu>(tx, tw, y, m, inter, k, ldy, st)
   switch (bn) {
-    case 256: return launch_gemm2<256, bf16, true>(tx, tw, y, m, inter, k, ldy, st, glu_limit);
-    case 128: return launch_gemm2<128, bf16, true>(tx, tw, y, m, inter, k, ldy, st, glu_limit);
-    default: return launch_gemm2<64, bf16, true>(tx, tw, y, m, inter, k, ldy, st, glu_limit);
+    NVLLM_G2G(256);
+    NVLLM_G2G(128);
+    default:
+      NVLLM_G2G(64);
   }
+#undef NVLLM_G2G
 }
 
 }  // namespace nvllm
