@@ -756,6 +756,9 @@ int launch_recurrence(const RecArgs& a, int n_seqs, cudaStream_t st) {
   if (a.dk <= 16) return launch_recurrence_as<16, 1, 2, CHD>(a, n_seqs, st);
   if (a.dk <= 32) return launch_recurrence_as<32, 1, 2, CHD>(a, n_seqs, st);
   if (a.dk <= 64) return launch_recurrence_as<32, 2, 2, CHD>(a, n_seqs, st);
+  // few (head, sequence) pairs with three staged rows per token: twice the lanes per column keep more warps in flight (one
+  // prompt of 4096 tokens, 16 heads: 1.39 vs 1.77 ms; 8 x 1024 tokens: 0.67 vs 0.64 ms)
+  if (CHD && a.dk > 64 && a.dk <= 128 && static_cast<int64_t>(a.heads) * n_seqs * 2 <= sm_count()) return launch_recurrence_as<16, 8, 2, CHD>(a, n_seqs, st);
   if (a.dk <= 128) return launch_recurrence_as<32, 4, 2, CHD>(a, n_seqs, st);
   if (a.dk <= 256) return launch_recurrence_as<32, 8, 2, CHD>(a, n_seqs, st);
   return launch_recurrence_as<32, 16, 2, CHD>(a, n_seqs, st);
