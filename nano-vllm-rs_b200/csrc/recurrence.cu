@@ -425,40 +425,43 @@ __global__ void __launch_bounds__(256) delta_prepare_vec_kernel(const DeltaPrepA
 }
 
 // out[t, c] = sigmoid(sum_r w2[r, c] x[t, r] + b[c])^(1 / tau) = exp(log sigmoid(z) / tau): the second step of a two-step projection,
-// its bias and the decay in one pass, all f32.  CTA = 16 tokens x 128 channels: the tokens' inner values in shared memory,
-// a thread per channel (w2 is stored [rank, channels]: coalesced), every weight read serves 16 tokens.
-constexpr int kLrTok = 16, kLrRank = 64;
+// its bias and the decay in one pass, all f32.  CTA = TOK tokens x 128 channels: the tokens' inner values in shared memory,
+// a thread per channel (w2 is stored [rank, channels]: coalesced), every weight read serves TOK tokens.
+constexpr int kLrRank = 64;
+template <int TOK>
 __global__ void __launch_bounds__(128) low_rank_decay_kernel(float* __restrict__ out, int64_t ldo, const float* __restrict__ x, int64_t ldx,
                                                              const float* __restrict__ w2, const float* __restrict__ bias, int n, int rank,
                                                              int channels, float inv_tau) {
-  __shared__ float xs[kLrRank][kLrTok];
-  const int c = blockIdx.x * 128 + threadIdx.x, t0 = blockIdx.y * kLrTok, cnt = min(kLrTok, n - t0);
-  float acc[kLrTok];
+  __shared__ float xs[kLrRank][TOK];
+  const int c = blockIdx.x * 128 + threadIdx.x, t0 = blockIdx.y * TOK, cnt = min(TOK, n - t0);
+  float acc[TOK];
 #pragma unroll
-  for (int t = 0; t < kLrTok; ++t) acc[t] = 0.f;
+  for (int t = 0; t < TOK; ++t) acc[t] = 0.f;
   for (int r0 = 0; r0 < rank; r0 += kLrRank) {
     const int rc = min(kLrRank, rank - r0);
     __syncthreads();
-    for (int e = threadIdx.x; e < kLrTok * rc; e += 128) {
+    for (int e = threadIdx.x; e < TOK * rc; e += 128) {
       const int t = e / rc, r = e - t * rc;
       xs[r][t] = t < cnt ? x[(t0 + t) * ldx + r0 + r] : 0.f;
     }
     __syncthreads();
     if (c < channels) {
+#pragma unroll 8
       for (int r = 0; r < rc; ++r) {
         const float w = w2[static_cast<int64_t>(r0 + r) * channels + c];
 #pragma unroll
-        for (int t = 0; t < kLrTok; ++t) acc[t] = fmaf(w, xs[r][t], acc[t]);
+        for (int t = 0; t < TOK; ++t) acc[t] = fmaf(w, xs[r][t], acc[t]);
       }
     }
   }
   if (c >= channels) return;
   const float b = bias ? bias[c] : 0.f;
 #pragma unroll
-  for (int t = 0; t < kLrTok; ++t) {
+  for (int t = 0; t < TOK; ++t) {
     if (t >= cnt) break;
     const float z = acc[t] + b;
-    out[(t0 + t) * ldo + c] = expf((fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * inv_tau);
+    // (the inner exponential's relative error grows with |z| no faster than its share of the sum shrinks)
+    out[(t0 + t) * ldo + c] = expf((fminf(z, 0.f) - log1pf(__expf(-fabsf(z)))) * inv_tau);
   }
 }
 
@@ -849,8 +852,12 @@ extern "C" int nvllm_low_rank_decay(float* out, int64_t ldo, const float* x, int
                   "low_rank_decay: n=%d rank=%d channels=%d tau=%g", n, rank, channels, tau);
   if (n == 0) return 0;
   NVLLM_CHECK_ARG(out && x && w2, NVLLM_ERR_ARG, "low_rank_decay: NULL");
-  dim3 grid((channels + 127) / 128, (n + kLrTok - 1) / kLrTok);
-  low_rank_decay_kernel<<<grid, 128, 0, static_cast<cudaStream_t>(stream)>>>(out, ldo, x, ldx, w2, bias, n, rank, channels, 1.0f / tau);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const int cols = (channels + 127) / 128;
+  if (static_cast<int64_t>(cols) * ((n + 15) / 16) >= 4 * sm_count())
+    low_rank_decay_kernel<16><<<dim3(cols, (n + 15) / 16), 128, 0, st>>>(out, ldo, x, ldx, w2, bias, n, rank, channels, 1.0f / tau);
+  else   // few tokens: more, shorter CTAs
+    low_rank_decay_kernel<4><<<dim3(cols, (n + 3) / 4), 128, 0, st>>>(out, ldo, x, ldx, w2, bias, n, rank, channels, 1.0f / tau);
   NVLLM_LAUNCH_CHECK("low_rank_decay_kernel");
   return 0;
 }

@@ -344,7 +344,7 @@ def test_padding_sequences_touch_no_state(cuda, kind):
     np.testing.assert_array_equal(npf(state), st0)
 
 
-@pytest.mark.parametrize("rank,ch,n,tau", [(4, 18, 7, 8.0), (16, 192, 33, 16.0), (1, 1, 1, 1.0), (70, 130, 16, 0.5), (130, 129, 17, 3.0)])
+@pytest.mark.parametrize("rank,ch,n,tau", [(4, 18, 7, 8.0), (20, 192, 33, 16.0), (1, 1, 1, 1.0), (70, 130, 16, 0.5), (130, 129, 17, 3.0), (12, 1024, 1500, 4.0), (70, 900, 1203, 2.0)])
 def test_low_rank_decay(cuda, rank, ch, n, tau):
     from nano_vllm_rs_b200 import ops
     rng = np.random.default_rng(rank)
