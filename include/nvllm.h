@@ -662,6 +662,68 @@ int nvllm_gemm_glu_bf16(void* out, const void* x, const void* w_gate_up, int32_t
 int nvllm_gemm_glu_bf16_grouped(void* y, const void* x, const void* w, int32_t max_rows, int32_t inter, int32_t k, int32_t groups,
                                 int64_t ldx, int64_t ldw, int64_t ldy, const int32_t* tile_group, float limit, void* stream);
 
+/* ---- Capped scores with a slope per head, keys in two parts, YaRN rotary, element-wise output gates, gelu gates, experts that
+ * scale their input, per-layer token inputs ------------------------------------------------------------------------------- */
+
+/* nvllm_masked_attention with two more options, each off when NULL / 0:
+ *   slopes (f32 [heads]): slopes[h] * (p - j) is taken off the score of key j, after the cap (excludes dist_bias).  With a cap, keys so
+ *     far back that their weight is exactly zero in f32 are not read;
+ *   shared_dim > 0: a key of dim values is [dim - shared_dim values of its head, k_cache row (kv_heads x (dim - shared_dim)) |
+ *     shared_dim values that all heads share, row `slot` of k_shared, rows ks_row apart]. */
+int nvllm_extended_attention(void* out, int64_t ldo, const void* q, int64_t ldq, const float* gate, int64_t ldg,
+                             int32_t gate_per_head, const void* k_cache, const void* v_cache, int64_t k_row, int64_t v_row,
+                             const int32_t* tok_seq, const int64_t* positions, const int32_t* block_tables, int32_t table_cap,
+                             int32_t block_size, int32_t n, int32_t heads, int32_t kv_heads, int32_t dim, int32_t vdim, float scale,
+                             float softcap, float temp_coef, int32_t temp_every, int32_t window, int32_t keep_first,
+                             const float* sinks, int32_t chunk, const float* head_scale, const float* dist_bias, int32_t dist_rows,
+                             const float* out_rot_table, int32_t max_pos, const float* slopes, const void* k_shared, int64_t ks_row,
+                             int32_t shared_dim, const int32_t* cu_tokens, int32_t n_seqs, int32_t dtype, void* stream);
+/* nvllm_rope_table_interleaved with YaRN scaling: with dim(t) = dims ln(original / (2 pi t)) / (2 ln base), lo = max(floor(dim(fast)), 0),
+ * hi = min(ceil(dim(slow)), dims - 1) and r_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), pair i turns by
+ * f_i / factor r_i + f_i (1 - r_i) per position, and cos and sin carry the factor 0.1 ln(factor) + 1. */
+int nvllm_rope_table_yarn(float* cos_sin, int32_t max_pos, int32_t dims, double base, double factor, double fast, double slow,
+                          double original, void* stream);
+/* Latent attention, per-token preparation from f32 projection rows: cq[t] = rms(proj[t, :q_rank]) * dq_norm_w;
+ * cache row slots[t] (slot < 0: none) and dense row t (nullable) = [rms(proj[t, kv_off : kv_off + kv_rank]) * c_norm_w | the next rot_dim
+ * values, the first rot_dims of them rotated (pairs (2i, 2i+1))], rows cache_row apart. */
+int nvllm_latent_norm_store(void* cq, int64_t ldcq, const float* proj, int64_t ldp, int32_t q_rank, const float* dq_norm_w, int32_t kv_off,
+                            int32_t kv_rank, int32_t rot_dim, const float* c_norm_w, float eps, const int64_t* positions,
+                            const float* rope_table, int32_t rot_dims, int32_t max_pos, void* cache, void* dense, int64_t cache_row,
+                            const int32_t* slots, int32_t n, int32_t dtype, void* stream);
+/* In place on rows of heads x [dim | rot_dim]: the first rot_dims of every head's last rot_dim values are rotated (pairs (2i, 2i+1)). */
+int nvllm_rotate_tail(void* x, int64_t ldx, const int64_t* positions, const float* rope_table, int32_t rot_dims, int32_t max_pos, int32_t n,
+                      int32_t heads, int32_t dim, int32_t rot_dim, int32_t dtype, void* stream);
+/* nvllm_linear times a gate: y[b][m, n] = (x[b] w[b]^T)[m, n] * sigmoid(gate[m * ldg + b * bsg + n]) (gate f32, nullable). */
+int nvllm_linear_gated(void* y, const void* x, const void* w, int32_t m, int32_t n, int32_t k, int64_t ldx, int64_t ldw,
+                       int64_t ldy, int32_t batch, int64_t bsx, int64_t bsw, int64_t bsy, const float* gate, int64_t ldg,
+                       int64_t bsg, int32_t dtype, int32_t out_dtype, void* stream);
+/* y[i, c] *= sigmoid(gate[i, c]) in place (gate f32). */
+int nvllm_sigmoid_gate(void* y, int64_t ldy, const float* gate, int64_t ldg, int32_t n, int32_t cols, int32_t dtype, void* stream);
+/* Gates of a feed-forward's pair of products.  (nvllm_ff_activation_params kind 3: gelu_tanh(in[i, c]) * in[i, ff + c].) */
+enum nvllm_gate { NVLLM_GATE_SILU = 1, NVLLM_GATE_CLAMPED = 2, NVLLM_GATE_GELU = 3 };
+/* nvllm_gemm_glu_bf16 / _grouped with the gate named (limit: the clamped gate's).  row_scale (f32 [max_rows], nullable, SiLU only): row r
+ * is the product of row_scale[r] * x[r] (applied to the f32 accumulators). */
+int nvllm_gemm_gated_bf16(void* out, const void* x, const void* w_gate_up, int32_t m, int32_t inter, int32_t k, int64_t ldx,
+                          int64_t ldw, int64_t ldout, int32_t gate, float limit, void* workspace, size_t workspace_bytes, void* stream);
+int nvllm_gemm_gated_bf16_grouped(void* y, const void* x, const void* w, int32_t max_rows, int32_t inter, int32_t k, int32_t groups,
+                                  int64_t ldx, int64_t ldw, int64_t ldy, const int32_t* tile_group, int32_t gate, float limit,
+                                  const float* row_scale, void* stream);
+/* nvllm_linear_grouped with a factor per row on its input (row_scale f32 [max_rows], nullable). */
+int nvllm_linear_grouped_scaled(void* y, const void* x, const void* w, int32_t max_rows, int32_t n, int32_t k, int64_t ldx, int64_t ldw,
+                                int64_t ldy, int64_t group_stride_w, const int32_t* row_src, const float* row_scale,
+                                const int32_t* tile_group, int32_t glu, float limit, int32_t dtype, int32_t out_dtype, void* stream);
+/* Routing on sigmoid scores: chosen = the `top` largest of logits + bias (bias nullable; ties: lowest index); topk_w = sigmoid of the
+ * chosen ones, as they are.  (nvllm_moe_combine with topk_w == NULL adds the expert outputs as they are.) */
+int nvllm_moe_route_sigmoid(int32_t* topk_idx, float* topk_w, const float* logits, int64_t ld, const float* bias, int32_t n,
+                            int32_t experts, int32_t top, void* stream);
+/* nvllm_moe_sort that also writes, beside every row, its assignment's weight (row_weight f32 [max_rows], nullable; padding rows: 0). */
+int nvllm_moe_sort_weighted(int32_t* row_token, float* row_weight, int32_t* tile_expert, int32_t* slot_row, const int32_t* topk_idx,
+                            const float* topk_w, int32_t n, int32_t top, int32_t experts, int32_t max_rows, int32_t tile_rows,
+                            void* stream);
+/* out[t, c] = gelu_tanh(gate[t, c]) * table[ids[t], col0 + c], c < dim (gate f32; table and out in `dtype`; ids clamped to the table). */
+int nvllm_token_gate(void* out, const float* gate, int64_t ldg, const void* table, int64_t ld_table, int64_t col0, const int64_t* ids,
+                     int32_t vocab, int32_t n, int32_t dim, int32_t dtype, void* stream);
+
 /* ------------------------------------------------------------------------------------------------
  * Engine-level C ABI: the C++ host runtime that mirrors the reference's Rust types one-to-one
  * (Config, SamplingParams, Sequence, BlockManager, Scheduler, ModelRunner, Qwen3Model, LLMEngine).

@@ -139,6 +139,19 @@ PROTOTYPES = {
     "nvllm_low_rank_decay": (i32, [vp, i64, vp, i64, vp, vp, i32, i32, i32, f32, vp]),
     "nvllm_gemm_glu_bf16": (i32, [vp, vp, vp, i32, i32, i32, i64, i64, i64, f32, vp, sz, vp]),
     "nvllm_gemm_glu_bf16_grouped": (i32, [vp, vp, vp, i32, i32, i32, i32, i64, i64, i64, vp, f32, vp]),
+    "nvllm_extended_attention": (i32, [vp, i64, vp, i64, vp, i64, i32, vp, vp, i64, i64, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32,
+                                       f32, f32, f32, i32, i32, i32, vp, i32, vp, vp, i32, vp, i32, vp, vp, i64, i32, vp, i32, i32, vp]),
+    "nvllm_rope_table_yarn": (i32, [vp, i32, i32, f64, f64, f64, f64, f64, vp]),
+    "nvllm_latent_norm_store": (i32, [vp, i64, vp, i64, i32, vp, i32, i32, i32, vp, f32, vp, vp, i32, i32, vp, vp, i64, vp, i32, i32, vp]),
+    "nvllm_rotate_tail": (i32, [vp, i64, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp]),
+    "nvllm_linear_gated": (i32, [vp, vp, vp, i32, i32, i32, i64, i64, i64, i32, i64, i64, i64, vp, i64, i64, i32, i32, vp]),
+    "nvllm_sigmoid_gate": (i32, [vp, i64, vp, i64, i32, i32, i32, vp]),
+    "nvllm_gemm_gated_bf16": (i32, [vp, vp, vp, i32, i32, i32, i64, i64, i64, i32, f32, vp, sz, vp]),
+    "nvllm_gemm_gated_bf16_grouped": (i32, [vp, vp, vp, i32, i32, i32, i32, i64, i64, i64, vp, i32, f32, vp, vp]),
+    "nvllm_linear_grouped_scaled": (i32, [vp, vp, vp, i32, i32, i32, i64, i64, i64, i64, vp, vp, vp, i32, f32, i32, i32, vp]),
+    "nvllm_moe_route_sigmoid": (i32, [vp, vp, vp, i64, vp, i32, i32, i32, vp]),
+    "nvllm_moe_sort_weighted": (i32, [vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, vp]),
+    "nvllm_token_gate": (i32, [vp, vp, i64, vp, i64, i64, vp, i32, i32, i32, i32, vp]),
 }
 
 

@@ -6,7 +6,9 @@
 //   * an optional sliding window: position p sees the keys p - window + 1 .. p   (window <= 0: all keys 0 .. p),
 //     and, with keep > 0, the first `keep` keys of its sequence whatever their distance,
 //   * optional sinks: a learned number per head whose exponential joins the softmax denominator (no key, no value),
-//   * the gate as one number per head instead of one per output value.
+//   * the gate as one number per head instead of one per output value,
+//   * a slope per head: slope_h * (p - j) is taken off the (capped) score of key j,
+//   * keys in two parts: per-head values, and values that all heads of a token share.
 // Every query token carries its sequence (a row of the block tables) and its position, so one launch serves whole prompts,
 // portions of prompts and single decoded tokens side by side; position p sees the keys 0..p of its sequence.
 //
@@ -40,6 +42,23 @@ __global__ void attn_bias_store_kernel(T* __restrict__ q, int64_t ldq, T* __rest
   if (slot < 0) return;
   for (int c = threadIdx.x; c < kn; c += blockDim.x) stv(kc + slot * k_row + c, p[qn + c] + (kb ? kb[c] : 0.f));
   for (int c = threadIdx.x; c < vn; c += blockDim.x) stv(vc + slot * v_row + c, p[qn + kn + c] + (vb ? vb[c] : 0.f));
+}
+
+// The same without biases, in 16-byte steps: every size a multiple of 4, aligned rows.
+template <typename T>
+__global__ void __launch_bounds__(256) attn_store_vec_kernel(T* __restrict__ q, int64_t ldq, T* __restrict__ kc, T* __restrict__ vc, int64_t k_row, int64_t v_row,
+                                                             const float* __restrict__ proj, int64_t ldp, const int32_t* __restrict__ slots, int qn, int kn, int vn) {
+  const int64_t t = blockIdx.x;
+  const float4* p = reinterpret_cast<const float4*>(proj + t * ldp);
+  const int32_t slot = slots[t];
+  const int end = (slot < 0 ? qn : qn + kn + vn) / 4;
+  for (int c = threadIdx.x; c < end; c += blockDim.x) {
+    const float4 v = p[c];
+    const int e = 4 * c;
+    T* dst = e < qn ? q + t * ldq + e : (e < qn + kn ? kc + slot * k_row + (e - qn) : vc + slot * v_row + (e - qn - kn));
+    if (sizeof(T) == 2) *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
+    else *reinterpret_cast<float4*>(dst) = v;
+  }
 }
 
 // The same step for layers whose queries and keys are RMS-normed over the WHOLE projection (all heads of a token at once,
@@ -453,6 +472,8 @@ struct AttnArgs {
   const float2* out_rot;     // [max_pos, vdim / 2] (cos, sin): every head's output is turned by -p, value m paired with m + vdim / 2
   int max_pos;
   int bias_staged;           // tensor-core kernel: the CTA copies its heads' rows of dist_bias into shared memory first
+  const float* slopes;       // [heads]: slopes[h] * (p - j) is taken off the score of key j, after the cap
+  const void* ks; int64_t ks_row; int shared;   // shared > 0: the last `shared` values of every head's key are row `slot` of ks
 };
 
 // shared memory the tensor-core kernel may spend on the distance-bias rows of a CTA's heads (two CTAs per SM still fit)
@@ -463,6 +484,13 @@ __device__ __forceinline__ int first_key(const AttnArgs& a, int p) {
   int lo = a.window > 0 ? max(0, p - a.window + 1) : 0;
   if (a.chunk > 0) lo = max(lo, p / a.chunk * a.chunk);
   return lo;
+}
+
+// With a cap and a slope the keys further back than this carry exactly no weight: scores lie within +-cap before the slope, so a
+// key d tokens back is at least slope d - 2 cap below the row's own key, and exp(-104) is below the smallest f32 number.
+__device__ __forceinline__ int slope_first_key(const AttnArgs& a, int p, float slope) {
+  const float reach = (2.0f * a.softcap + 104.0f) / slope;
+  return a.softcap > 0.f && slope > 0.f && reach < static_cast<float>(p) ? p - static_cast<int>(reach) - 1 : 0;
 }
 
 constexpr int kMaxVPerLane = 16;  // vdim <= 512
@@ -486,13 +514,15 @@ __global__ void __launch_bounds__(128) capped_attn_warp_kernel(const AttnArgs a)
   __syncwarp();
   const int32_t* table = a.tables ? a.tables + static_cast<int64_t>(a.tok_seq[t]) * a.table_cap : nullptr;
   const int64_t dense0 = a.dense_cu ? a.dense_cu[a.tok_seq[t]] : 0;
-  const T* kc = static_cast<const T*>(a.kc) + static_cast<int64_t>(g) * a.dim;
+  const int own = a.dim - a.shared;   // values of a key that are the head's own
+  const T* kc = static_cast<const T*>(a.kc) + static_cast<int64_t>(g) * own;
   const T* vc = static_cast<const T*>(a.vc) + static_cast<int64_t>(g) * a.vdim;
+  const float slope = a.slopes ? a.slopes[h] : 0.f;
   float m = -INFINITY, l = 0.f, acc[kMaxVPerLane];
 #pragma unroll
   for (int i = 0; i < kMaxVPerLane; ++i) acc[i] = 0.f;
   const int nkeys = static_cast<int>(pos) + 1;
-  const int first = first_key(a, static_cast<int>(pos));   // passes start at multiples of 32 whatever the window or chunk
+  const int first = max(first_key(a, static_cast<int>(pos)), slope_first_key(a, static_cast<int>(pos), slope));   // passes start at multiples of 32 whatever the window or chunk
   for (int j0 = a.keep > 0 ? 0 : first & ~31; j0 < nkeys; j0 += 32) {
     if (j0 >= a.keep && j0 < (first & ~31)) j0 = first & ~31;   // past the kept keys: on to the window
     const int j = j0 + lane;
@@ -504,8 +534,13 @@ __global__ void __launch_bounds__(128) capped_attn_warp_kernel(const AttnArgs a)
         slot = table ? static_cast<int64_t>(blk) * a.block_size + j % a.block_size : dense0 + j;
         const T* kr = kc + slot * a.k_row;
         float d = 0.f;
-        for (int c = 0; c < a.dim; ++c) d = fmaf(qw[c], ldv(kr + c), d);
+        for (int c = 0; c < own; ++c) d = fmaf(qw[c], ldv(kr + c), d);
+        if (a.shared > 0) {
+          const T* sr = static_cast<const T*>(a.ks) + slot * a.ks_row;
+          for (int c = 0; c < a.shared; ++c) d = fmaf(qw[own + c], ldv(sr + c), d);
+        }
         s = a.softcap > 0.f ? a.softcap * tanhf(d / a.softcap) : d;
+        if (a.slopes) s -= slope * static_cast<float>(nkeys - 1 - j);
         if (a.dist_bias) s += a.dist_bias[static_cast<int64_t>(h) * a.dist_rows + min(nkeys - 1 - j, a.dist_rows - 1)];
       }
     }
@@ -593,11 +628,14 @@ __device__ __forceinline__ float fast_tanh(float x) { return 1.0f - __fdividef(2
 
 // One warp's share of a key tile: 16 rows x (16 NP) keys -> S on tensor cores, cap / mask / online softmax in f32, then
 // O[:, 0 .. 16 VP) += P . V.  k_addr / v_addr are the warp's ldmatrix lane addresses of its first key (and first value column).
-// bias (EXT): per row, the row of the distance-bias table of the row's head (null: none), one value per distance.
-template <int DMAX, int VMAX, int NP, int VP, int QS, int VS, bool EXT>
+// bias (kExtTable): per row, the row of the distance-bias table of the row's head (null: none), one value per distance.
+// slope2 (kExtSlope): per row, the slope of the row's head in log2 units.
+enum { kExtNone = 0, kExtTable = 1, kExtSlope = 2 };
+template <int DMAX, int VMAX, int NP, int VP, int QS, int VS, int EXT>
 __device__ __forceinline__ void attn_tile(float (&o)[VMAX / 8][4], float (&m)[2], float (&l)[2], uint32_t q_addr, uint32_t k_addr,
                                           uint32_t v_addr, int key0, const int (&pos)[2], const int (&lo)[2], const float (&qscale)[2],
-                                          bool capped, float cap2, bool need_mask, int tq4, const float* const (&bias)[2], int dist_rows, int keep) {
+                                          bool capped, float cap2, bool need_mask, int tq4, const float* const (&bias)[2], int dist_rows, int keep,
+                                          const float (&slope2)[2]) {
   float s[2 * NP][4];
 #pragma unroll
   for (int i = 0; i < 2 * NP; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
@@ -614,14 +652,24 @@ __device__ __forceinline__ void attn_tile(float (&o)[VMAX / 8][4], float (&m)[2]
     }
   }
   float mx[2] = {-INFINITY, -INFINITY};
+  float b0[2];   // what the slope takes off this lane's first key; every further key costs one FMA
+  if (EXT == kExtSlope) {
+#pragma unroll
+    for (int i = 0; i < 2; ++i) b0[i] = -slope2[i] * static_cast<float>(pos[i] - key0 - 2 * tq4);
+  }
 #pragma unroll
   for (int nt = 0; nt < 2 * NP; ++nt)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int i = e >> 1, j = key0 + nt * 8 + 2 * tq4 + (e & 1);
       float v = s[nt][e] * qscale[i];            // with a cap: the score over the cap; without: the score in log2 units
-      if (capped) v = cap2 * fast_tanh(v);
-      if (EXT) { if (bias[i] != nullptr && j <= pos[i]) v = fmaf(bias[i][min(pos[i] - j, dist_rows - 1)], kLog2e, v); }
+      if (EXT == kExtSlope) {
+        const float b = fmaf(slope2[i], static_cast<float>(nt * 8 + (e & 1)), b0[i]);
+        v = capped ? fmaf(cap2, fast_tanh(v), b) : v + b;
+      } else if (capped) {
+        v = cap2 * fast_tanh(v);
+      }
+      if (EXT == kExtTable) { if (bias[i] != nullptr && j <= pos[i]) v = fmaf(bias[i][min(pos[i] - j, dist_rows - 1)], kLog2e, v); }
       if (need_mask) v = (j <= pos[i] && (j >= lo[i] || j < keep)) ? v : -INFINITY;   // lo: the first key of the row's window or chunk
       s[nt][e] = v;
       mx[i] = fmaxf(mx[i], v);
@@ -665,8 +713,8 @@ __device__ __forceinline__ void attn_tile(float (&o)[VMAX / 8][4], float (&m)[2]
   }
 }
 
-template <int DMAX, int VMAX, bool EXT>
-__global__ void __launch_bounds__(kThreads, 2) capped_attn_mma_kernel(const AttnArgs a, const int32_t* __restrict__ cu_tokens, int n_seqs, int tq,
+template <int DMAX, int VMAX, int EXT>
+__global__ void __launch_bounds__(kThreads, DMAX > 128 ? 1 : 2) capped_attn_mma_kernel(const AttnArgs a, const int32_t* __restrict__ cu_tokens, int n_seqs, int tq,
                                                               int group) {
   constexpr int QS = DMAX + 8, VS = VMAX + 8;       // shared-memory row strides (elements): 16-byte rows, conflict-free ldmatrix
   extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -691,17 +739,18 @@ __global__ void __launch_bounds__(kThreads, 2) capped_attn_mma_kernel(const Attn
   const int32_t* table = a.tables ? a.tables + static_cast<int64_t>(seq) * a.table_cap : nullptr;
   const int64_t dense0 = cu_tokens[seq];
   const bf16* qg = static_cast<const bf16*>(a.q);
-  const bf16* kc = static_cast<const bf16*>(a.kc) + static_cast<int64_t>(g) * a.dim;
+  const bf16* kc = static_cast<const bf16*>(a.kc) + static_cast<int64_t>(g) * (a.dim - a.shared);
+  const bf16* ks = static_cast<const bf16*>(a.ks);
   const bf16* vc = static_cast<const bf16*>(a.vc) + static_cast<int64_t>(g) * a.vdim;
   // zero everything once (padding columns and rows stay zero), then the query rows
   for (int i = tid; i < (kRows * QS + 2 * kKeys * QS + 2 * kKeys * VS) / 8; i += kThreads) reinterpret_cast<uint4*>(smem_raw)[i] = make_uint4(0, 0, 0, 0);
   // the distance-bias rows of this CTA's heads (consecutive rows of the table), behind the tiles: one shared-memory load per
   // score instead of a global one
   float* bias_s = reinterpret_cast<float*>(smem_raw + static_cast<size_t>(kRows * QS + 2 * kKeys * QS + 2 * kKeys * VS) * sizeof(bf16));
-  if (EXT && a.bias_staged)
+  if (EXT == kExtTable && a.bias_staged)
     for (int i = tid; i < group * a.dist_rows; i += kThreads) bias_s[i] = a.dist_bias[static_cast<int64_t>(g) * group * a.dist_rows + i];
   __syncthreads();
-  const int dch = a.dim / 8, vch = a.vdim / 8;     // 16-byte chunks per row
+  const int dch = a.dim / 8, och = (a.dim - a.shared) / 8, vch = a.vdim / 8;     // 16-byte chunks per row (och: a key's own part)
   // the query rows travel with the first key tile's copy group (asynchronous: no thread waits for its own row here)
   for (int i = tid; i < kRows * dch; i += kThreads) {
     const int r = i / dch, c = i % dch, t = r / group, hr = r % group;
@@ -729,7 +778,11 @@ __global__ void __launch_bounds__(kThreads, 2) capped_attn_mma_kernel(const Attn
     const bf16* ksrc = slot >= 0 ? kc + slot * a.k_row : kc;
     const bf16* vsrc = slot >= 0 ? vc + slot * a.v_row : vc;
     const int nb = slot >= 0 ? 16 : 0;
-    for (int c = lh; c < dch; c += 4) cp_async_16(smem_u32(kd + c * 8), ksrc + (nb ? c * 8 : 0), nb);
+    for (int c = lh; c < och; c += 4) cp_async_16(smem_u32(kd + c * 8), ksrc + (nb ? c * 8 : 0), nb);
+    if (och < dch) {   // the part that all heads share
+      const bf16* ssrc = slot >= 0 ? ks + slot * a.ks_row : ks;
+      for (int c = lh; c < dch - och; c += 4) cp_async_16(smem_u32(kd + (och + c) * 8), ssrc + (nb ? c * 8 : 0), nb);
+    }
     for (int c = lh; c < vch; c += 4) cp_async_16(smem_u32(vd + c * 8), vsrc + (nb ? c * 8 : 0), nb);
     cp_async_commit();
   };
@@ -740,6 +793,11 @@ __global__ void __launch_bounds__(kThreads, 2) capped_attn_mma_kernel(const Attn
   const int rbase = few ? 0 : warp * 16, kq = warp & 3, vh = warp >> 2;
   int pos[2], lo[2]; float qscale[2]; bool valid[2];
   const float* bias[2] = {nullptr, nullptr};
+  float slope2[2] = {0.f, 0.f}, slope_min = 0.f;
+  if (EXT == kExtSlope) {   // the group's smallest slope decides how far back the CTA has to look
+    slope_min = a.slopes[g * group];
+    for (int h = 1; h < group; ++h) slope_min = fminf(slope_min, a.slopes[g * group + h]);
+  }
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     const int r = rbase + gq + 8 * i, t = r / group;
@@ -748,10 +806,11 @@ __global__ void __launch_bounds__(kThreads, 2) capped_attn_mma_kernel(const Attn
     lo[i] = valid[i] ? first_key(a, pos[i]) : -(1 << 30);   // a row sees the keys lo .. pos
     qscale[i] = a.scale * (1.0f + a.temp_coef * logf(floorf(static_cast<float>((pos[i] + 1) / a.temp_every)) + 1.0f)) *
                 (a.softcap > 0.f ? 1.0f / a.softcap : kLog2e);
-    if (EXT) {
+    if (EXT != kExtNone) {
       const int h = g * group + r % group;
       if (a.head_scale) qscale[i] *= a.head_scale[h];
-      if (a.dist_bias) bias[i] = a.bias_staged ? bias_s + (r % group) * a.dist_rows : a.dist_bias + static_cast<int64_t>(h) * a.dist_rows;
+      if (EXT == kExtSlope) slope2[i] = a.slopes[h] * kLog2e;
+      else if (a.dist_bias) bias[i] = a.bias_staged ? bias_s + (r % group) * a.dist_rows : a.dist_bias + static_cast<int64_t>(h) * a.dist_rows;
     }
   }
   // the smallest position of the warp's rows decides whether a tile needs the causal mask (empty rows count as hidden)
@@ -767,7 +826,8 @@ __global__ void __launch_bounds__(kThreads, 2) capped_attn_mma_kernel(const Attn
   const int ntiles = (nkeys + kKeys - 1) / kKeys;
   // with a window the first tile is the one that holds the first key the CTA's first token sees (tiles stay anchored at
   // multiples of 64 from the sequence's start)
-  const int kt0 = first_key(a, static_cast<int>(a.positions[tok0])) / kKeys;   // (windows and chunks only move forward with the position)
+  const int p0 = static_cast<int>(a.positions[tok0]);
+  const int kt0 = max(first_key(a, p0), EXT == kExtSlope ? slope_first_key(a, p0, slope_min) : 0) / kKeys;   // (all of them only move forward with the position)
   // the tiles of the kept first keys come before the window's; tile number `it` of the walk is key tile tile_of(it)
   const int nkeep = min((a.keep + kKeys - 1) / kKeys, kt0), iters = nkeep + ntiles - kt0;
   auto tile_of = [&](int it) { return it < nkeep ? it : it - nkeep + kt0; };
@@ -789,7 +849,7 @@ __global__ void __launch_bounds__(kThreads, 2) capped_attn_mma_kernel(const Attn
       if (key0 < nkeys && (it >= nkeep || key0 < a.keep))
         attn_tile<DMAX, VMAX, 1, VMAX / 32, QS, VS, EXT>(o, m, l, q_addr, smem_u32(kb + kq * 16 * QS + k_lane),
                                                          smem_u32(vb + kq * 16 * VS + vh * (VMAX / 2) + v_lane), key0, pos, lo, qscale, capped, cap2,
-                                                         key0 + 15 > min_pos || key0 < max_lo, tq4, bias, a.dist_rows, a.keep);
+                                                         key0 + 15 > min_pos || key0 < max_lo, tq4, bias, a.dist_rows, a.keep, slope2);
     } else if (warp_has_rows) {
       // two halves of 32 keys: half the score registers of a 64-key pass (no spills under the 128-register cap)
 #pragma unroll
@@ -797,7 +857,7 @@ __global__ void __launch_bounds__(kThreads, 2) capped_attn_mma_kernel(const Attn
         if (it < nkeep && kt * kKeys + hf * 32 >= a.keep) break;   // nothing kept in this half
         attn_tile<DMAX, VMAX, 2, VMAX / 16, QS, VS, EXT>(o, m, l, q_addr, smem_u32(kb + hf * 32 * QS + k_lane), smem_u32(vb + hf * 32 * VS + v_lane),
                                                          kt * kKeys + hf * 32, pos, lo, qscale, capped, cap2,
-                                                         kt * kKeys + hf * 32 + 31 > min_pos || kt * kKeys + hf * 32 < max_lo, tq4, bias, a.dist_rows, a.keep);
+                                                         kt * kKeys + hf * 32 + 31 > min_pos || kt * kKeys + hf * 32 < max_lo, tq4, bias, a.dist_rows, a.keep, slope2);
       }
     }
     if (tid < kKeys) slot_s[buf][tid] = slot_ahead;   // this tile's slots were consumed by its load_tile an iteration ago
@@ -899,14 +959,14 @@ __global__ void __launch_bounds__(kThreads, 2) capped_attn_mma_kernel(const Attn
   }
 }
 
-template <int DMAX, int VMAX, bool EXT>
+template <int DMAX, int VMAX, int EXT>
 int launch_mma(AttnArgs a, const int32_t* cu_tokens, int n_seqs, cudaStream_t st) {
   const int group = a.heads / a.kv_heads, tq = kRows / group;
   const size_t tiles = (static_cast<size_t>(kRows) * (DMAX + 8) + 2 * kKeys * (DMAX + 8) + 2 * kKeys * (VMAX + 8)) * sizeof(bf16);
   const size_t bias_bytes = static_cast<size_t>(group) * a.dist_rows * sizeof(float);
-  a.bias_staged = EXT && a.dist_bias != nullptr && bias_bytes <= kBiasSmemBytes;
+  a.bias_staged = EXT == kExtTable && a.dist_bias != nullptr && bias_bytes <= kBiasSmemBytes;
   const size_t smem = tiles + (a.bias_staged ? bias_bytes : 0);
-  NVLLM_SMEM_ATTR_ONCE((capped_attn_mma_kernel<DMAX, VMAX, EXT>), tiles + (EXT ? kBiasSmemBytes : 0));
+  NVLLM_SMEM_ATTR_ONCE((capped_attn_mma_kernel<DMAX, VMAX, EXT>), tiles + (EXT == kExtTable ? kBiasSmemBytes : 0));
   dim3 grid((a.n + tq - 1) / tq + n_seqs, a.kv_heads);
   capped_attn_mma_kernel<DMAX, VMAX, EXT><<<grid, kThreads, smem, st>>>(a, cu_tokens, n_seqs, tq, group);
   NVLLM_LAUNCH_CHECK("capped_attn_mma_kernel");
@@ -928,6 +988,17 @@ extern "C" int nvllm_attn_bias_store(void* q, int64_t ldq, void* k_cache, void* 
   if (n == 0) return 0;
   NVLLM_CHECK_ARG(q && k_cache && v_cache && proj && slots, NVLLM_ERR_ARG, "attn_bias_store: NULL");
   cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (!q_bias && !k_bias && !v_bias && q_cols % 4 == 0 && k_cols % 4 == 0 && v_cols % 4 == 0 && ldq % 4 == 0 && k_row % 4 == 0 && v_row % 4 == 0 &&
+      ldp % 4 == 0 && aligned16(q) && aligned16(k_cache) && aligned16(v_cache) && aligned16(proj)) {
+    if (dtype == NVLLM_BF16)
+      attn_store_vec_kernel<bf16><<<n, 256, 0, st>>>(static_cast<bf16*>(q), ldq, static_cast<bf16*>(k_cache), static_cast<bf16*>(v_cache), k_row, v_row, proj,
+                                                     ldp, slots, q_cols, k_cols, v_cols);
+    else
+      attn_store_vec_kernel<float><<<n, 256, 0, st>>>(static_cast<float*>(q), ldq, static_cast<float*>(k_cache), static_cast<float*>(v_cache), k_row, v_row,
+                                                      proj, ldp, slots, q_cols, k_cols, v_cols);
+    NVLLM_LAUNCH_CHECK("attn_store_vec_kernel");
+    return 0;
+  }
   if (dtype == NVLLM_BF16)
     attn_bias_store_kernel<bf16><<<n, 256, 0, st>>>(static_cast<bf16*>(q), ldq, static_cast<bf16*>(k_cache), static_cast<bf16*>(v_cache), k_row,
                                                     v_row, proj, ldp, q_bias, k_bias, v_bias, slots, q_cols, k_cols, v_cols);
@@ -1094,6 +1165,23 @@ extern "C" int nvllm_masked_attention(void* out, int64_t ldo, const void* q, int
                                       int32_t keep_first, const float* sinks, int32_t chunk, const float* head_scale,
                                       const float* dist_bias, int32_t dist_rows, const float* out_rot_table, int32_t max_pos,
                                       const int32_t* cu_tokens, int32_t n_seqs, int32_t dtype, void* stream) {
+  return nvllm_extended_attention(out, ldo, q, ldq, gate, ldg, gate_per_head, k_cache, v_cache, k_row, v_row, tok_seq, positions, block_tables,
+                                  table_cap, block_size, n, heads, kv_heads, dim, vdim, scale, softcap, temp_coef, temp_every, window, keep_first, sinks,
+                                  chunk, head_scale, dist_bias, dist_rows, out_rot_table, max_pos, nullptr, nullptr, 0, 0, cu_tokens, n_seqs, dtype, stream);
+}
+
+extern "C" int nvllm_extended_attention(void* out, int64_t ldo, const void* q, int64_t ldq, const float* gate, int64_t ldg,
+                                        int32_t gate_per_head, const void* k_cache, const void* v_cache, int64_t k_row, int64_t v_row,
+                                        const int32_t* tok_seq, const int64_t* positions, const int32_t* block_tables,
+                                        int32_t table_cap, int32_t block_size, int32_t n, int32_t heads, int32_t kv_heads, int32_t dim,
+                                        int32_t vdim, float scale, float softcap, float temp_coef, int32_t temp_every, int32_t window,
+                                        int32_t keep_first, const float* sinks, int32_t chunk, const float* head_scale,
+                                        const float* dist_bias, int32_t dist_rows, const float* out_rot_table, int32_t max_pos,
+                                        const float* slopes, const void* k_shared, int64_t ks_row, int32_t shared_dim,
+                                        const int32_t* cu_tokens, int32_t n_seqs, int32_t dtype, void* stream) {
+  NVLLM_CHECK_ARG(shared_dim >= 0 && shared_dim < dim && (shared_dim == 0 || (k_shared != nullptr && ks_row >= shared_dim)) &&
+                      (slopes == nullptr || dist_bias == nullptr), NVLLM_ERR_ARG,
+                  "attention: %d of %d key values shared by the heads; a slope per head excludes a distance table", shared_dim, dim);
   NVLLM_CHECK_ARG(chunk >= 0 && keep_first >= 0 && (dist_bias == nullptr || dist_rows > 0) && (out_rot_table == nullptr || (max_pos > 0 && vdim % 2 == 0)),
                   NVLLM_ERR_ARG, "attention: chunk=%d dist_rows=%d max_pos=%d vdim=%d (an output rotation pairs the halves of an even vdim)", chunk,
                   dist_rows, max_pos, vdim);
@@ -1105,27 +1193,29 @@ extern "C" int nvllm_masked_attention(void* out, int64_t ldo, const void* q, int
   NVLLM_CHECK_ARG(out && q && k_cache && v_cache && tok_seq && positions && (block_tables || cu_tokens), NVLLM_ERR_ARG, "attention: NULL");
   AttnArgs a{out, ldo, q, ldq, gate, ldg, k_cache, v_cache, k_row, v_row, tok_seq, positions, block_tables, table_cap, block_size,
              n, heads, kv_heads, dim, vdim, scale, softcap, temp_coef, temp_every, window > 0 ? window : 0, sinks, gate_per_head, block_tables ? nullptr : cu_tokens,
-             keep_first, chunk, head_scale, dist_bias, dist_rows, reinterpret_cast<const float2*>(out_rot_table), max_pos, 0};
+             keep_first, chunk, head_scale, dist_bias, dist_rows, reinterpret_cast<const float2*>(out_rot_table), max_pos, 0,
+             slopes, k_shared, ks_row, shared_dim};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   // bf16 with 16-byte rows and a token range per sequence: tensor cores; everything else (f32, odd sizes): one warp per row
   const int group = heads / kv_heads;
   if (dtype == NVLLM_BF16 && cu_tokens != nullptr && n_seqs > 0 && knobs().capped_mma && group <= kRows && dim % 8 == 0 && vdim % 8 == 0 &&
-      dim <= 128 && vdim <= 128 && ldq % 8 == 0 && k_row % 8 == 0 && v_row % 8 == 0 && ldo % 2 == 0 && aligned16(q) && aligned16(k_cache) &&
+      dim <= 192 && vdim <= 128 && shared_dim % 8 == 0 && ks_row % 8 == 0 && aligned16(k_shared) && ldq % 8 == 0 && k_row % 8 == 0 && v_row % 8 == 0 && ldo % 2 == 0 && aligned16(q) && aligned16(k_cache) &&
       aligned16(v_cache) && (reinterpret_cast<uintptr_t>(out) & 3u) == 0) {
     // the factor per head and the distance bias live in a second instantiation, so that kernels without them keep their
     // registers (the output rotation only touches the epilogue)
-    const bool ext = head_scale != nullptr || dist_bias != nullptr;
+    const int ext = slopes != nullptr ? kExtSlope : (head_scale != nullptr || dist_bias != nullptr) ? kExtTable : kExtNone;
     const int vmax = vdim <= 64 ? 64 : 128;
     // the output rotation pairs column c with c + vdim / 2 inside one thread's accumulators: vdim must fill the tile
-    if (out_rot_table == nullptr || (vdim == vmax && aligned16(out_rot_table))) {
-      if (!ext) {
-        if (dim <= 64 && vdim <= 64) return launch_mma<64, 64, false>(a, cu_tokens, n_seqs, st);
-        if (vdim <= 64) return launch_mma<128, 64, false>(a, cu_tokens, n_seqs, st);
-        return launch_mma<128, 128, false>(a, cu_tokens, n_seqs, st);
-      }
-      if (dim <= 64 && vdim <= 64) return launch_mma<64, 64, true>(a, cu_tokens, n_seqs, st);
-      if (vdim <= 64) return launch_mma<128, 64, true>(a, cu_tokens, n_seqs, st);
-      return launch_mma<128, 128, true>(a, cu_tokens, n_seqs, st);
+    if ((out_rot_table == nullptr || (vdim == vmax && aligned16(out_rot_table))) && (dim <= 128 || ext == kExtNone)) {
+#define NVLLM_ATTN(EXTV)                                                                              \
+  if (dim <= 64 && vdim <= 64) return launch_mma<64, 64, EXTV>(a, cu_tokens, n_seqs, st);             \
+  if (vdim <= 64) return launch_mma<128, 64, EXTV>(a, cu_tokens, n_seqs, st);                         \
+  return launch_mma<128, 128, EXTV>(a, cu_tokens, n_seqs, st)
+      if (dim > 128) return launch_mma<192, 128, kExtNone>(a, cu_tokens, n_seqs, st);
+      if (ext == kExtNone) { NVLLM_ATTN(kExtNone); }
+      if (ext == kExtSlope) { NVLLM_ATTN(kExtSlope); }
+      NVLLM_ATTN(kExtTable);
+#undef NVLLM_ATTN
     }
   }
   const unsigned grid = static_cast<unsigned>((static_cast<int64_t>(n) * heads + 3) / 4);

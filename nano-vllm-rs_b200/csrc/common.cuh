@@ -166,13 +166,27 @@ __device__ __forceinline__ float glu_clamped_fast(float g, float u, float limit)
   g = fminf(g, limit);
   return __fdividef(g, 1.0f + __expf(-1.702f * g)) * (fminf(fmaxf(u, -limit), limit) + 1.0f);
 }
+// silu where a bf16 result follows: fast exponential and division (the division's divisor must stay below 2^126).
+__device__ __forceinline__ float silu_fast(float g) { return __fdividef(g, 1.0f + __expf(fminf(-g, 80.0f))); }
+// The tanh form of gelu, 0.5 z (1 + tanh(a)) with a = sqrt(2 / pi) (z + 0.044715 z^3), written as z sigmoid(2 a): one exponential,
+// saturating cleanly at both ends.
+constexpr float kGeluA = 1.5957691216057308f;   // 2 sqrt(2 / pi)
+__device__ __forceinline__ float gelu_tanh(float z) { return z / (1.0f + expf(-kGeluA * fmaf(0.044715f * z * z, z, z))); }
+// The same where a bf16 result follows.
+__device__ __forceinline__ float gelu_tanh_fast(float z) {
+  const float e = __expf(fminf(-kGeluA * fmaf(0.044715f * z * z, z, z), 80.0f));
+  return __fdividef(z, 1.0f + e);
+}
 // One pair of a gated feed-forward's activations from bf16 pre-activations (gb: two gates, ub: two ups) in a GEMM epilogue.
-// GATE 1: silu(g) u, silu rounded to bf16 (the rounding points of a separate activation kernel); GATE 2: the clamped gate.
-enum { kGateNone = 0, kGateSilu = 1, kGateClamped = 2 };
+// GATE 1: silu(g) u, silu rounded to bf16 (the rounding points of a separate activation kernel); GATE 2: the clamped gate;
+// GATE 3: gelu_tanh(g) u; GATE 4: silu(g) u of rows that carry a factor on their input (the epilogue multiplies it in first).
+enum { kGateNone = 0, kGateSilu = 1, kGateClamped = 2, kGateGelu = 3, kGateSiluRow = 4 };
 template <int GATE>
 __device__ __forceinline__ float2 gated_pair(uint32_t gb, uint32_t ub, float limit) {
   const float g0 = bf16_lo(gb), g1 = bf16_hi(gb);
   if (GATE == kGateClamped) return make_float2(glu_clamped_fast(g0, bf16_lo(ub), limit), glu_clamped_fast(g1, bf16_hi(ub), limit));
+  if (GATE == kGateGelu) return make_float2(gelu_tanh_fast(g0) * bf16_lo(ub), gelu_tanh_fast(g1) * bf16_hi(ub));
+  if (GATE == kGateSiluRow) return make_float2(silu_fast(g0) * bf16_lo(ub), silu_fast(g1) * bf16_hi(ub));
   const uint32_t sb = pack_bf16x2(g0 / (1.0f + expf(-g0)), g1 / (1.0f + expf(-g1)));
   return make_float2(bf16_lo(sb) * bf16_lo(ub), bf16_hi(sb) * bf16_hi(ub));
 }

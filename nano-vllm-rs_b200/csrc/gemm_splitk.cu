@@ -381,17 +381,19 @@ namespace nvllm {
 #endif
 
 int gemm_splitk_dispatch(void* y, const void* x, const void* w, int m, int n, int k, int64_t ldx, int64_t ldw, int64_t ldy,
-                         bool gated, int bn, int sk, cudaStream_t st, const RowPush& ps, float glu_limit) {
+                         int gate, int bn, int sk, cudaStream_t st, const RowPush& ps, float glu_limit) {
   CUtensorMap tx, tw;
+  const bool gated = gate != kGateNone;
   const int n_acc = gated ? 2 * n : n;
   if (int rc = make_tmap_bf16_2d(&tx, x, m, k, ldx, 128)) return rc;
   if (int rc = make_tmap_bf16_2d(&tw, w, n_acc, k, ldw, gated ? bn / 2 : bn)) return rc;
   const int mt = (m + 127) / 128, tiles = mt * (n_acc / bn);
 #define NVLLM_SK(BNV, SKV)                                                                                   \
   if (bn == BNV && sk == SKV)                                                                                \
-    return !gated           ? launch_splitk<BNV, SKV, kGateNone>(tx, tw, y, m, n, k, ldy, tiles, mt, st, ps)                        \
-           : glu_limit > 0.f ? launch_splitk<BNV, SKV, kGateClamped>(tx, tw, y, m, n, k, ldy, tiles, mt, st, RowPush{}, glu_limit) \
-                             : launch_splitk<BNV, SKV, kGateSilu>(tx, tw, y, m, n, k, ldy, tiles, mt, st, RowPush{})
+    return !gated                 ? launch_splitk<BNV, SKV, kGateNone>(tx, tw, y, m, n, k, ldy, tiles, mt, st, ps)                       \
+           : gate == kGateClamped ? launch_splitk<BNV, SKV, kGateClamped>(tx, tw, y, m, n, k, ldy, tiles, mt, st, RowPush{}, glu_limit) \
+           : gate == kGateGelu    ? launch_splitk<BNV, SKV, kGateGelu>(tx, tw, y, m, n, k, ldy, tiles, mt, st, RowPush{})               \
+                                  : launch_splitk<BNV, SKV, kGateSilu>(tx, tw, y, m, n, k, ldy, tiles, mt, st, RowPush{})
   NVLLM_SK(256, 8); NVLLM_SK(256, 4); NVLLM_SK(256, 2);
   NVLLM_SK(128, 8); NVLLM_SK(128, 4); NVLLM_SK(128, 2);
   NVLLM_SK(64, 4); NVLLM_SK(64, 2);

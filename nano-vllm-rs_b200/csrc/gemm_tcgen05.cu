@@ -74,7 +74,7 @@ __device__ __forceinline__ void store_row32<float>(float* dst, const uint32_t (&
 }
 
 // GATE != kGateNone: w = [gate (N rows) | up (N rows)]; the B tile is staged as BN/2 gate rows + the matching BN/2 up rows and
-// the epilogue writes y[:, n_tile*BN/2 + c] = silu(gate) * up, or with glu_limit > 0 the clamped gate of gated_pair (see gemm_tcgen05_2cta.cu for the CTA-pair variant).
+// the epilogue writes y[:, n_tile*BN/2 + c] = silu(gate) * up, or another gate of gated_pair (see gemm_tcgen05_2cta.cu for the CTA-pair variant).
 // Optional qkv epilogue (ROPE mode, BN == 128 == head_dim): each output tile is one head of the packed [q | k | v] row,
 // and each epilogue thread owns that head for one token.  It applies what Qwen3Attention::forward does between qkv_proj
 // and Attention::forward (qwen3.rs:219-229) plus Attention::store_kv_cache (attention.rs:150-174): round to bf16 (the
@@ -101,7 +101,8 @@ __global__ void __launch_bounds__(256, 1)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_constant__ CUtensorMap tmap_w,
                     OutT* __restrict__ y, int M, int N, int K, int64_t ldy, int num_m_tiles, int num_tiles,
                     const RopeEpi re = RopeEpi{}, int STAGES = GemmCfg<BN>::kStages, const RowPush ps = RowPush{},
-                    const int32_t* __restrict__ tile_group = nullptr, int group_rows = 0, float glu_limit = 0.f) {
+                    const int32_t* __restrict__ tile_group = nullptr, int group_rows = 0, float glu_limit = 0.f,
+                    const float* __restrict__ row_scale = nullptr) {
   // tile_group != nullptr (expert layers): 128-row tile m uses the weight block of group tile_group[m], i.e. rows
   // [group * group_rows, ...) of w; an unused tile (group < 0) runs against group 0 and its rows are never read.
   using C = GemmCfg<BN>;  // STAGES <= C::kStages: ring depth of this launch (fewer stages -> two CTAs per SM, see launch_gemm)
@@ -299,12 +300,18 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_con
           }
         }
       } else if constexpr (GATE != kGateNone) {
+        float rs = 1.0f;   // the factor on this row's input (both products are linear in it)
+        if constexpr (GATE == kGateSiluRow) rs = row < M ? row_scale[row] : 0.f;
 #pragma unroll 1
         for (int c = 0; c < BN / 64; ++c) {
           uint32_t g[32], u[32];
           tmem_ld_32x32b_x32(taddr + c * 32, g);
           tmem_ld_32x32b_x32(taddr + BN / 2 + c * 32, u);
           tmem_ld_wait();
+          if constexpr (GATE == kGateSiluRow) {
+#pragma unroll
+            for (int e = 0; e < 32; ++e) { g[e] = __float_as_uint(__uint_as_float(g[e]) * rs); u[e] = __float_as_uint(__uint_as_float(u[e]) * rs); }
+          }
 #pragma unroll
           for (int e = 0; e < 32; e += 2) {  // rounding points of the unfused path: bf16 gate_up, bf16 silu(gate)
             const uint32_t gb = pack_bf16x2(__uint_as_float(g[e]), __uint_as_float(g[e + 1]));
@@ -350,7 +357,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_con
 template <int BN, typename OutT, int GATE = kGateNone, int CN = 1, bool ROPE = false>
 static int launch_gemm(const CUtensorMap& tx, const CUtensorMap& tw, void* y, int M, int N, int K, int64_t ldy,
                        cudaStream_t st, const RopeEpi& re = RopeEpi{}, const RowPush& ps = RowPush{},
-                       const int32_t* tile_group = nullptr, int group_rows = 0, float glu_limit = 0.f) {
+                       const int32_t* tile_group = nullptr, int group_rows = 0, float glu_limit = 0.f, const float* row_scale = nullptr) {
   using C = GemmCfg<BN>;
   auto kern = gemm_tcgen05_kernel<BN, OutT, GATE, CN, ROPE>;
   NVLLM_SMEM_ATTR_ONCE(kern, C::kSmemBytes);
@@ -370,7 +377,7 @@ static int launch_gemm(const CUtensorMap& tx, const CUtensorMap& tw, void* y, in
   const int smem = C::kSmemBytes - (C::kStages - stages) * C::kStageBytes;
   if constexpr (CN == 1) {
     NVLLM_CUDA(launch_pdl(kern, dim3(clusters), dim3(256), smem, st, tx, tw, static_cast<OutT*>(y), M, N, K, ldy,
-                          num_m_tiles, num_tiles, re, stages, ps, tile_group, group_rows, glu_limit));
+                          num_m_tiles, num_tiles, re, stages, ps, tile_group, group_rows, glu_limit, row_scale));
   } else {
     cudaLaunchConfig_t cfg{};
     cfg.gridDim = dim3(clusters * CN);
@@ -385,15 +392,16 @@ static int launch_gemm(const CUtensorMap& tx, const CUtensorMap& tw, void* y, in
     cfg.attrs = attr;
     cfg.numAttrs = pdl_enabled() ? 2 : 1;
     NVLLM_CUDA(cudaLaunchKernelEx(&cfg, kern, tx, tw, static_cast<OutT*>(y), M, N, K, ldy, num_m_tiles, num_tiles, re,
-                                  static_cast<int>(C::kStages), ps, tile_group, group_rows, glu_limit));
+                                  static_cast<int>(C::kStages), ps, tile_group, group_rows, glu_limit, row_scale));
   }
   return 0;
 }
 
 template <int BN>
-static int launch_gated(const CUtensorMap& tx, const CUtensorMap& tw, void* y, int m, int inter, int k, int64_t ldy, float limit, cudaStream_t st,
+static int launch_gated(const CUtensorMap& tx, const CUtensorMap& tw, void* y, int m, int inter, int k, int64_t ldy, int gate, float limit, cudaStream_t st,
                         const int32_t* tile_group = nullptr) {
-  if (limit > 0.f) return launch_gemm<BN, bf16, kGateClamped>(tx, tw, y, m, inter, k, ldy, st, RopeEpi{}, RowPush{}, tile_group, 2 * inter, limit);
+  if (gate == kGateClamped) return launch_gemm<BN, bf16, kGateClamped>(tx, tw, y, m, inter, k, ldy, st, RopeEpi{}, RowPush{}, tile_group, 2 * inter, limit);
+  if (gate == kGateGelu) return launch_gemm<BN, bf16, kGateGelu>(tx, tw, y, m, inter, k, ldy, st, RopeEpi{}, RowPush{}, tile_group, 2 * inter);
   return launch_gemm<BN, bf16, kGateSilu>(tx, tw, y, m, inter, k, ldy, st, RopeEpi{}, RowPush{}, tile_group, 2 * inter);
 }
 
@@ -429,12 +437,12 @@ int gemm_2cta_dispatch(void* y, const void* x, const void* w, int m, int n, int 
                        int64_t ldy, int out_dtype, cudaStream_t st);  // gemm_tcgen05_2cta.cu
 
 int gemm_silu_2cta_dispatch(void* y, const void* x, const void* w, int m, int inter, int k, int64_t ldx, int64_t ldw,
-                            int64_t ldy, float glu_limit, cudaStream_t st);  // gemm_tcgen05_2cta.cu
+                            int64_t ldy, int gate, float glu_limit, cudaStream_t st);  // gemm_tcgen05_2cta.cu
 
 // gemm_splitk.cu: cluster split-K for decode-sized projections (m <= 256)
 bool splitk_choose(int m, int n_acc, int k, bool silu, int bn_default, int* out_bn, int* out_sk);
 int gemm_splitk_dispatch(void* y, const void* x, const void* w, int m, int n, int k, int64_t ldx, int64_t ldw, int64_t ldy,
-                         bool silu, int bn, int sk, cudaStream_t st, const RowPush& ps = RowPush{}, float glu_limit = 0.f);
+                         int gate, int bn, int sk, cudaStream_t st, const RowPush& ps = RowPush{}, float glu_limit = 0.f);
 
 static bool use_2cta();
 // CTA pairs pay off once there are at least two 256-row tiles or the problem is large enough to fill the machine with
@@ -483,7 +491,7 @@ int gemm_bf16_impl(void* y, const void* x, const void* w, int32_t m, int32_t n, 
   if (out_dtype == NVLLM_BF16) {  // decode-sized, long-K projections: split K over a cluster (gemm_splitk.cu)
     int sbn = 0, ssk = 0;
     if (splitk_choose(m, n, k, false, pick_bn(m, n), &sbn, &ssk))
-      return gemm_splitk_dispatch(y, x, w, m, n, k, ldx, ldw, ldy, false, sbn, ssk, st, ps);
+      return gemm_splitk_dispatch(y, x, w, m, n, k, ldx, ldw, ldy, kGateNone, sbn, ssk, st, ps);
   }
   if (!push && want_2cta(m, n, k)) return gemm_2cta_dispatch(y, x, w, m, n, k, ldx, ldw, ldy, out_dtype, st);
   const int bn = pick_bn(m, n);
@@ -550,7 +558,16 @@ extern "C" int nvllm_gemm_bf16_grouped(void* y, const void* x, const void* w, in
 extern "C" int nvllm_gemm_glu_bf16_grouped(void* y, const void* x, const void* w, int32_t max_rows, int32_t inter, int32_t k,
                                            int32_t groups, int64_t ldx, int64_t ldw, int64_t ldy, const int32_t* tile_group,
                                            float limit, void* stream) {
+  return nvllm_gemm_gated_bf16_grouped(y, x, w, max_rows, inter, k, groups, ldx, ldw, ldy, tile_group, limit > 0.f ? NVLLM_GATE_CLAMPED : NVLLM_GATE_SILU,
+                                       limit, nullptr, stream);
+}
+
+extern "C" int nvllm_gemm_gated_bf16_grouped(void* y, const void* x, const void* w, int32_t max_rows, int32_t inter, int32_t k,
+                                             int32_t groups, int64_t ldx, int64_t ldw, int64_t ldy, const int32_t* tile_group,
+                                             int32_t gate, float limit, const float* row_scale, void* stream) {
   using namespace nvllm;
+  NVLLM_CHECK_ARG(gate == NVLLM_GATE_SILU || (gate == NVLLM_GATE_CLAMPED && limit > 0.f && row_scale == nullptr) || (gate == NVLLM_GATE_GELU && row_scale == nullptr),
+                  NVLLM_ERR_ARG, "gemm_gated_grouped: gate %d, limit %g (a factor per row goes with SiLU)", gate, static_cast<double>(limit));
   NVLLM_CHECK_ARG(max_rows >= 0 && max_rows % 128 == 0 && inter > 0 && k > 0 && groups > 0 && k % 64 == 0 && inter % 64 == 0, NVLLM_ERR_ARG,
                   "gemm_glu_grouped: max_rows=%d (multiple of 128) inter=%d (%% 64) k=%d (%% 64) groups=%d", max_rows, inter, k, groups);
   NVLLM_CHECK_ARG(ldx >= k && ldw >= k && ldy >= inter && ldx % 8 == 0 && ldw % 8 == 0 && ldy % 8 == 0, NVLLM_ERR_ALIGN,
@@ -562,8 +579,11 @@ extern "C" int nvllm_gemm_glu_bf16_grouped(void* y, const void* x, const void* w
   CUtensorMap tx, tw;
   if (int rc = make_tmap_bf16_2d(&tx, x, max_rows, k, ldx, 128)) return rc;
   if (int rc = make_tmap_bf16_2d(&tw, w, static_cast<int64_t>(groups) * 2 * inter, k, ldw, bn / 2)) return rc;
-  if (bn == 256) return launch_gated<256>(tx, tw, y, max_rows, inter, k, ldy, limit, st, tile_group);
-  return launch_gated<128>(tx, tw, y, max_rows, inter, k, ldy, limit, st, tile_group);
+  if (row_scale != nullptr)
+    return bn == 256 ? launch_gemm<256, bf16, kGateSiluRow>(tx, tw, y, max_rows, inter, k, ldy, st, RopeEpi{}, RowPush{}, tile_group, 2 * inter, 0.f, row_scale)
+                     : launch_gemm<128, bf16, kGateSiluRow>(tx, tw, y, max_rows, inter, k, ldy, st, RopeEpi{}, RowPush{}, tile_group, 2 * inter, 0.f, row_scale);
+  if (bn == 256) return launch_gated<256>(tx, tw, y, max_rows, inter, k, ldy, gate, limit, st, tile_group);
+  return launch_gated<128>(tx, tw, y, max_rows, inter, k, ldy, gate, limit, st, tile_group);
 }
 
 // MergedColumnParallelLinear::forward + SiluAndMul::forward in one call (linear.rs:437-439 + activation.rs:46-63).
@@ -573,11 +593,20 @@ extern "C" int nvllm_gemm_silu_mul_bf16(void* out, const void* x, const void* w_
   return nvllm_gemm_glu_bf16(out, x, w_gate_up, m, inter, k, ldx, ldw, ldout, 0.f, workspace, workspace_bytes, stream);
 }
 
-// The same with the gate as a parameter: limit <= 0 SiLU, limit > 0 the clamped gate (gated_pair, common.cuh).
+// The same with the gate as a parameter (gated_pair, common.cuh).
 extern "C" int nvllm_gemm_glu_bf16(void* out, const void* x, const void* w_gate_up, int32_t m, int32_t inter, int32_t k,
                                    int64_t ldx, int64_t ldw, int64_t ldout, float limit, void* workspace,
                                    size_t workspace_bytes, void* stream) {
+  return nvllm_gemm_gated_bf16(out, x, w_gate_up, m, inter, k, ldx, ldw, ldout, limit > 0.f ? NVLLM_GATE_CLAMPED : NVLLM_GATE_SILU, limit, workspace,
+                               workspace_bytes, stream);
+}
+
+extern "C" int nvllm_gemm_gated_bf16(void* out, const void* x, const void* w_gate_up, int32_t m, int32_t inter, int32_t k,
+                                     int64_t ldx, int64_t ldw, int64_t ldout, int32_t gate, float limit, void* workspace,
+                                     size_t workspace_bytes, void* stream) {
   using namespace nvllm;
+  NVLLM_CHECK_ARG(gate == NVLLM_GATE_SILU || (gate == NVLLM_GATE_CLAMPED && limit > 0.f) || gate == NVLLM_GATE_GELU, NVLLM_ERR_ARG,
+                  "gemm_gated: gate %d, limit %g", gate, static_cast<double>(limit));
   NVLLM_CHECK_ARG(m >= 0 && inter > 0 && k > 0 && k % 64 == 0 && inter % 8 == 0, NVLLM_ERR_ARG,
                   "gemm_silu_mul: m=%d inter=%d k=%d (k %% 64, inter %% 8)", m, inter, k);
   NVLLM_CHECK_ARG(ldx >= k && ldw >= k && ldout >= inter && ldx % 8 == 0 && ldw % 8 == 0 && ldout % 8 == 0,
@@ -592,17 +621,17 @@ extern "C" int nvllm_gemm_glu_bf16(void* out, const void* x, const void* w_gate_
     {
       int sbn = 0, ssk = 0;
       if (splitk_choose(m, 2 * inter, k, true, bn, &sbn, &ssk))
-        return gemm_splitk_dispatch(out, x, w_gate_up, m, inter, k, ldx, ldw, ldout, true, sbn, ssk, st, RowPush{}, limit);
+        return gemm_splitk_dispatch(out, x, w_gate_up, m, inter, k, ldx, ldw, ldout, gate, sbn, ssk, st, RowPush{}, limit);
     }
-    if (want_2cta(m, 2 * inter, k)) return gemm_silu_2cta_dispatch(out, x, w_gate_up, m, inter, k, ldx, ldw, ldout, limit, st);
+    if (want_2cta(m, 2 * inter, k)) return gemm_silu_2cta_dispatch(out, x, w_gate_up, m, inter, k, ldx, ldw, ldout, gate, limit, st);
     CUtensorMap tx, tw;
     if (int rc = make_tmap_bf16_2d(&tx, x, m, k, ldx, 128)) return rc;
     if (int rc = make_tmap_bf16_2d(&tw, w_gate_up, 2 * static_cast<int64_t>(inter), k, ldw, bn / 2)) return rc;
     switch (bn) {
-      case 256: return launch_gated<256>(tx, tw, out, m, inter, k, ldout, limit, st);
-      case 192: return launch_gated<192>(tx, tw, out, m, inter, k, ldout, limit, st);
-      case 128: return launch_gated<128>(tx, tw, out, m, inter, k, ldout, limit, st);
-      default: return launch_gated<64>(tx, tw, out, m, inter, k, ldout, limit, st);
+      case 256: return launch_gated<256>(tx, tw, out, m, inter, k, ldout, gate, limit, st);
+      case 192: return launch_gated<192>(tx, tw, out, m, inter, k, ldout, gate, limit, st);
+      case 128: return launch_gated<128>(tx, tw, out, m, inter, k, ldout, gate, limit, st);
+      default: return launch_gated<64>(tx, tw, out, m, inter, k, ldout, gate, limit, st);
     }
   }
   // odd intermediate sizes: plain GEMM into the workspace, then the SiLU*mul kernel
@@ -611,7 +640,8 @@ extern "C" int nvllm_gemm_glu_bf16(void* out, const void* x, const void* w_gate_
                   "gemm_silu_mul: workspace %zu < %zu bytes", workspace_bytes, need);
   NVLLM_CHECK_ARG(ldout == inter, NVLLM_ERR_ARG, "gemm_silu_mul: unfused path needs a contiguous output");
   if (int rc = nvllm_gemm_bf16(workspace, x, w_gate_up, m, 2 * inter, k, ldx, ldw, 2 * inter, NVLLM_BF16, nullptr, 0, stream)) return rc;
-  if (limit > 0.f) return nvllm_glu_clamped(out, workspace, m, inter, limit, NVLLM_BF16, stream);
+  if (gate == kGateClamped) return nvllm_glu_clamped(out, workspace, m, inter, limit, NVLLM_BF16, stream);
+  if (gate == kGateGelu) return nvllm_ff_activation_params(out, workspace, m, inter, 3, nullptr, NVLLM_BF16, stream);
   return nvllm_silu_mul(out, workspace, m, inter, NVLLM_BF16, stream);
 }
 

@@ -49,7 +49,7 @@ __device__ __forceinline__ void store_row32_2(OutT* dst, const uint32_t (&r)[32]
 // GATE != kGateNone: w is the packed [gate (N rows) | up (N rows)] matrix of MergedColumnParallelLinear (linear.rs:421-433);
 // the leader CTA stages BN/2 gate rows, its peer the matching BN/2 up rows, so accumulator columns [0, BN/2) are gate and
 // [BN/2, BN) are up for the same BN/2 output features, and the epilogue writes y[:, n_tile*BN/2 + c] = silu(gate)*up
-// (SiluAndMul::forward, activation.rs:46-63; glu_limit > 0: the clamped gate of gated_pair) without the [M, 2N] intermediate ever reaching HBM.  N = output features.
+// (SiluAndMul::forward, activation.rs:46-63; or another gate of gated_pair) without the [M, 2N] intermediate ever reaching HBM.  N = output features.
 template <int BN, typename OutT, int GATE>
 __global__ void __launch_bounds__(256, 1)
 gemm_tcgen05_2cta_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_constant__ CUtensorMap tmap_w,
@@ -261,9 +261,9 @@ int gemm_2cta_dispatch(void* y, const void* x, const void* w, int m, int n, int 
 #undef NVLLM_G2
 }
 
-// y[M, inter] = silu(x . Wgate^T) * (x . Wup^T) (or the clamped gate) with w = [Wgate | Wup] packed row-wise ([2*inter, K]).
+// y[M, inter] = silu(x . Wgate^T) * (x . Wup^T) (or another gate) with w = [Wgate | Wup] packed row-wise ([2*inter, K]).
 int gemm_silu_2cta_dispatch(void* y, const void* x, const void* w, int m, int inter, int k, int64_t ldx, int64_t ldw,
-                            int64_t ldy, float glu_limit, cudaStream_t st) {
+                            int64_t ldy, int gate, float glu_limit, cudaStream_t st) {
   // accumulator tile BN covers BN/2 output features; reuse the tile heuristic on the 2*inter accumulator columns
   const int bn = pick_bn_2cta(m, 2 * inter);
   NVLLM_CHECK_ARG(inter % (bn / 2) == 0 || true, NVLLM_ERR_ARG, "gemm_silu: inter");
@@ -272,8 +272,9 @@ int gemm_silu_2cta_dispatch(void* y, const void* x, const void* w, int m, int in
   if (int rc = make_tmap_bf16_2d(&tw, w, 2 * static_cast<int64_t>(inter), k, ldw, bn / 2)) return rc;
 #define NVLLM_G2G(BNV)                                                                                                    \
   case BNV:                                                                                                               \
-    return glu_limit > 0.f ? launch_gemm2<BNV, bf16, kGateClamped>(tx, tw, y, m, inter, k, ldy, st, glu_limit)            \
-                           : launch_gemm2<BNV, bf16, kGateSilu>(tx, tw, y, m, inter, k, ldy, st)
+    return gate == kGateClamped ? launch_gemm2<BNV, bf16, kGateClamped>(tx, tw, y, m, inter, k, ldy, st, glu_limit)       \
+           : gate == kGateGelu  ? launch_gemm2<BNV, bf16, kGateGelu>(tx, tw, y, m, inter, k, ldy, st)                     \
+                                : launch_gemm2<BNV, bf16, kGateSilu>(tx, tw, y, m, inter, k, ldy, st)
   switch (bn) {
     NVLLM_G2G(256);
     NVLLM_G2G(128);

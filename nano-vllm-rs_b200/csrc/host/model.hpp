@@ -73,5 +73,6 @@ ModelImpl* make_talapel(const json::Value& cfg);  // talapel_model.cu
 ModelImpl* make_zudatar(const json::Value& cfg);  // zudatar_model.cu
 ModelImpl* make_zasorax(const json::Value& cfg);  // zasorax_model.cu
 ModelImpl* make_kalesun(const json::Value& cfg);  // kalesun_model.cu
+ModelImpl* make_fomerax(const json::Value& cfg);  // fomerax_model.cu
 
 }  // namespace nvllm

@@ -15,6 +15,8 @@
 // Options of the attention (nvllm_latent_window_attention): a sliding window (position p sees p - window + 1 .. p), a sink
 // per head whose exponential joins the softmax denominator, and a gate per head (out *= sigmoid(gate)); the rotated part
 // may be absent (rot_dim = 0).
+#include <cmath>
+
 #include "common.cuh"
 
 namespace nvllm {
@@ -51,6 +53,123 @@ __global__ void rope_table_interleaved_kernel(float2* __restrict__ tab, int max_
     }
     const double a = static_cast<double>(p) * f;
     tab[e] = make_float2(static_cast<float>(cos(a)), static_cast<float>(sin(a)));
+  }
+}
+
+// The YaRN form of the scaling: pair i's share of the slowed-down frequency f / factor is a linear ramp over the pair index from
+// lo (share 0) to hi (share 1); cos and sin are multiplied by `amp`.
+__global__ void rope_table_yarn_kernel(float2* __restrict__ tab, int max_pos, int half, int dims, double base, double factor, double lo, double hi, double amp) {
+  const int64_t total = static_cast<int64_t>(max_pos) * half;
+  for (int64_t e = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; e < total; e += static_cast<int64_t>(gridDim.x) * blockDim.x) {
+    const int64_t p = e / half;
+    const int i = static_cast<int>(e - p * half);
+    const double f = pow(base, -2.0 * i / dims);
+    const double r = fmin(fmax((i - lo) / fmax(hi - lo, 0.001), 0.0), 1.0);
+    const double a = static_cast<double>(p) * (f / factor * r + f * (1.0 - r));
+    tab[e] = make_float2(static_cast<float>(cos(a) * amp), static_cast<float>(sin(a) * amp));
+  }
+}
+
+// Everything between a latent layer's input projection and its query up-projection, one warp per (token, part), f32 in:
+//   part 0: rms(query latent) * dq_w -> cq;   part 1: rms(latent) * c_w and the rotated shared key part -> the token's cache row
+//   [latent | key part] (slot < 0: none) and, with `dense`, the same row in the step's own order.
+struct NormStoreArgs {
+  const float* proj; int64_t ldp; int kv_off;    // proj row: query latent at 0, [latent | key part] at kv_off
+  void* cq; int64_t ldcq; const float* dq_w;
+  void *cache, *dense; int64_t cache_row; const float* c_w;
+  const int64_t* positions; const float2* table; int rot_dims, max_pos;
+  const int32_t* slots;
+  int n, q_rank, kv_rank, rot_dim; float eps;
+};
+
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(128) latent_norm_store_kernel(const NormStoreArgs a) {
+  const int lane = threadIdx.x & 31;
+  const int64_t item = static_cast<int64_t>(blockIdx.x) * 4 + (threadIdx.x >> 5);
+  if (item >= 2 * static_cast<int64_t>(a.n)) return;
+  const int64_t t = item >> 1;
+  const bool kv = item & 1;
+  const int32_t slot = kv ? a.slots[t] : 0;
+  const float* src = a.proj + t * a.ldp + (kv ? a.kv_off : 0);
+  const float* w = kv ? a.c_w : a.dq_w;
+  const int cols = kv ? a.kv_rank : a.q_rank;
+  T* d0 = kv ? (slot >= 0 ? static_cast<T*>(a.cache) + slot * a.cache_row : nullptr) : static_cast<T*>(a.cq) + t * a.ldcq;
+  T* d1 = kv && a.dense ? static_cast<T*>(a.dense) + t * a.cache_row : nullptr;
+  if (d0 == nullptr && d1 == nullptr) return;
+  float ss = 0.f;
+  if (VEC) {
+    for (int c = 4 * lane; c < cols; c += 128) {
+      const float4 v = *reinterpret_cast<const float4*>(src + c);
+      ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
+  } else {
+    for (int c = lane; c < cols; c += 32) ss = fmaf(src[c], src[c], ss);
+  }
+  const float r = 1.0f / sqrtf(warp_sum(ss) / cols + a.eps);
+  auto put4 = [](T* p, const float4& o) {
+    if (sizeof(T) == 2) *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(o.x, o.y), pack_bf16x2(o.z, o.w));
+    else *reinterpret_cast<float4*>(p) = o;
+  };
+  if (VEC) {
+    for (int c = 4 * lane; c < cols; c += 128) {
+      const float4 v = *reinterpret_cast<const float4*>(src + c), ww = *reinterpret_cast<const float4*>(w + c);
+      const float4 o = make_float4(v.x * r * ww.x, v.y * r * ww.y, v.z * r * ww.z, v.w * r * ww.w);
+      if (d0) put4(d0 + c, o);
+      if (d1) put4(d1 + c, o);
+    }
+  } else {
+    for (int c = lane; c < cols; c += 32) {
+      const float o = src[c] * r * w[c];
+      if (d0) stf(d0 + c, o);
+      if (d1) stf(d1 + c, o);
+    }
+  }
+  if (!kv) return;
+  int64_t pos = a.positions[t];
+  pos = pos < 0 ? 0 : (pos >= a.max_pos ? a.max_pos - 1 : pos);
+  const float2* tab = a.table + pos * (a.rot_dims / 2);
+  for (int i = lane; i < a.rot_dim; i += 32) {
+    float v = src[cols + i];
+    if (i < a.rot_dims) {
+      const float2 cs = tab[i >> 1];
+      const float o = src[cols + (i ^ 1)];
+      v = (i & 1) ? fmaf(v, cs.x, o * cs.y) : fmaf(v, cs.x, -o * cs.y);   // (u cos - v sin, v cos + u sin)
+    }
+    if (d0) stf(d0 + cols + i, v);
+    if (d1) stf(d1 + cols + i, v);
+  }
+}
+
+// The rotated part of every query head in place: x rows of heads x [dim | rot_dim], pairs (2i, 2i + 1) of the first rot_dims values
+// behind dim.  A thread takes PAIRS neighbouring pairs of one head.
+template <typename T, int PAIRS>
+__global__ void __launch_bounds__(256) rotate_tail_kernel(T* __restrict__ x, int64_t ldx, const int64_t* __restrict__ positions, const float2* __restrict__ table,
+                                                          int max_pos, int64_t n, int heads, int dim, int rot_dim, int half) {
+  const int per = half / PAIRS;
+  const int64_t total = n * heads * per;
+  for (int64_t e = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; e < total; e += static_cast<int64_t>(gridDim.x) * blockDim.x) {
+    const int64_t th = e / per, t = th / heads;
+    const int i = static_cast<int>(e - th * per) * PAIRS, h = static_cast<int>(th - t * heads);
+    int64_t pos = positions[t];
+    pos = pos < 0 ? 0 : (pos >= max_pos ? max_pos - 1 : pos);
+    const float2* tab = table + pos * half + i;
+    T* p = x + t * ldx + static_cast<int64_t>(h) * (dim + rot_dim) + dim + 2 * i;
+    if (PAIRS == 4) {   // T is bf16 here: one 16-byte access
+      uint4 v = *reinterpret_cast<const uint4*>(p);
+      uint32_t* u = reinterpret_cast<uint32_t*>(&v);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const float2 cs = tab[k];
+        const float lo = bf16_lo(u[k]), hi = bf16_hi(u[k]);
+        u[k] = pack_bf16x2(fmaf(lo, cs.x, -hi * cs.y), fmaf(hi, cs.x, lo * cs.y));
+      }
+      *reinterpret_cast<uint4*>(p) = v;
+    } else {
+      const float u = ldf(p), v = ldf(p + 1);
+      const float2 cs = *tab;
+      stf(p, fmaf(u, cs.x, -v * cs.y));
+      stf(p + 1, fmaf(v, cs.x, u * cs.y));
+    }
   }
 }
 
@@ -594,6 +713,74 @@ extern "C" int nvllm_rope_table_scaled(float* cos_sin, int32_t max_pos, int32_t 
   rope_table_interleaved_kernel<<<static_cast<unsigned>(blocks), 256, 0, static_cast<cudaStream_t>(stream)>>>(
       reinterpret_cast<float2*>(cos_sin), max_pos, dims / 2, dims, base, RopeScaling{factor, low, high, original});
   NVLLM_LAUNCH_CHECK("rope_table_interleaved_kernel");
+  return 0;
+}
+
+extern "C" int nvllm_rope_table_yarn(float* cos_sin, int32_t max_pos, int32_t dims, double base, double factor, double fast, double slow,
+                                     double original, void* stream) {
+  NVLLM_CHECK_ARG(cos_sin && max_pos > 0 && dims > 0 && dims % 2 == 0 && base > 1.0 && factor > 0.0 && fast > 0.0 && slow > 0.0 && original > 0.0,
+                  NVLLM_ERR_ARG, "rope_table_yarn: max_pos=%d dims=%d (even) base=%g (> 1) factor=%g fast=%g slow=%g original=%g", max_pos, dims, base,
+                  factor, fast, slow, original);
+  // index of the pair whose wave turns `turns` times within `original` positions
+  auto index_at = [&](double turns) { return dims * std::log(original / (6.283185307179586476925 * turns)) / (2.0 * std::log(base)); };
+  const double lo = std::fmax(std::floor(index_at(fast)), 0.0), hi = std::fmin(std::ceil(index_at(slow)), dims - 1.0);
+  const int64_t total = static_cast<int64_t>(max_pos) * (dims / 2);
+  int64_t blocks = (total + 255) / 256;
+  if (blocks > sm_count() * 16) blocks = sm_count() * 16;
+  rope_table_yarn_kernel<<<static_cast<unsigned>(blocks), 256, 0, static_cast<cudaStream_t>(stream)>>>(
+      reinterpret_cast<float2*>(cos_sin), max_pos, dims / 2, dims, base, factor, lo, hi, 0.1 * std::log(factor) + 1.0);
+  NVLLM_LAUNCH_CHECK("rope_table_yarn_kernel");
+  return 0;
+}
+
+extern "C" int nvllm_latent_norm_store(void* cq, int64_t ldcq, const float* proj, int64_t ldp, int32_t q_rank, const float* dq_norm_w, int32_t kv_off,
+                                       int32_t kv_rank, int32_t rot_dim, const float* c_norm_w, float eps, const int64_t* positions,
+                                       const float* rope_table, int32_t rot_dims, int32_t max_pos, void* cache, void* dense, int64_t cache_row,
+                                       const int32_t* slots, int32_t n, int32_t dtype, void* stream) {
+  NVLLM_CHECK_ARG(n >= 0 && q_rank > 0 && kv_rank > 0 && rot_dim >= 0 && kv_off >= q_rank && ldcq >= q_rank && cache_row >= kv_rank + rot_dim &&
+                      ldp >= kv_off + kv_rank + rot_dim && max_pos > 0, NVLLM_ERR_ARG, "latent_norm_store: q_rank=%d kv_rank=%d rot_dim=%d", q_rank, kv_rank,
+                  rot_dim);
+  NVLLM_CHECK_ARG(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= rot_dim, NVLLM_ERR_ARG,
+                  "latent_norm_store: rot_dims=%d must be even and at most rot_dim=%d", rot_dims, rot_dim);
+  NVLLM_CHECK_ARG(dtype == NVLLM_BF16 || dtype == NVLLM_F32, NVLLM_ERR_DTYPE, "latent_norm_store: dtype %d", dtype);
+  if (n == 0) return 0;
+  NVLLM_CHECK_ARG(cq && proj && dq_norm_w && c_norm_w && positions && (rope_table || rot_dims == 0) && cache && slots, NVLLM_ERR_ARG, "latent_norm_store: NULL");
+  const NormStoreArgs a{proj, ldp, kv_off, cq, ldcq, dq_norm_w, cache, dense, cache_row, c_norm_w, positions, reinterpret_cast<const float2*>(rope_table),
+                        rot_dims, max_pos, slots, n, q_rank, kv_rank, rot_dim, eps};
+  const unsigned grid = static_cast<unsigned>((2 * static_cast<int64_t>(n) + 3) / 4);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const bool vec = q_rank % 4 == 0 && kv_rank % 4 == 0 && kv_off % 4 == 0 && ldp % 4 == 0 && ldcq % 4 == 0 && cache_row % 4 == 0 && aligned16(proj) &&
+                   aligned16(cq) && aligned16(cache) && aligned16(dense) && aligned16(dq_norm_w) && aligned16(c_norm_w);
+  if (dtype == NVLLM_BF16) {
+    if (vec) latent_norm_store_kernel<bf16, true><<<grid, 128, 0, st>>>(a);
+    else latent_norm_store_kernel<bf16, false><<<grid, 128, 0, st>>>(a);
+  } else {
+    if (vec) latent_norm_store_kernel<float, true><<<grid, 128, 0, st>>>(a);
+    else latent_norm_store_kernel<float, false><<<grid, 128, 0, st>>>(a);
+  }
+  NVLLM_LAUNCH_CHECK("latent_norm_store_kernel");
+  return 0;
+}
+
+extern "C" int nvllm_rotate_tail(void* x, int64_t ldx, const int64_t* positions, const float* rope_table, int32_t rot_dims, int32_t max_pos, int32_t n,
+                                 int32_t heads, int32_t dim, int32_t rot_dim, int32_t dtype, void* stream) {
+  NVLLM_CHECK_ARG(n >= 0 && heads > 0 && dim >= 0 && rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= rot_dim && max_pos > 0 &&
+                      ldx >= static_cast<int64_t>(heads) * (dim + rot_dim), NVLLM_ERR_ARG, "rotate_tail: heads=%d dim=%d rot_dim=%d rot_dims=%d (even)", heads,
+                  dim, rot_dim, rot_dims);
+  NVLLM_CHECK_ARG(dtype == NVLLM_BF16 || dtype == NVLLM_F32, NVLLM_ERR_DTYPE, "rotate_tail: dtype %d", dtype);
+  if (n == 0 || rot_dims == 0) return 0;
+  NVLLM_CHECK_ARG(x && positions && rope_table, NVLLM_ERR_ARG, "rotate_tail: NULL");
+  const bool vec = dtype == NVLLM_BF16 && rot_dims % 8 == 0 && dim % 8 == 0 && rot_dim % 8 == 0 && ldx % 8 == 0 && aligned16(x);
+  const int half = rot_dims / 2;
+  int64_t blocks = (static_cast<int64_t>(n) * heads * (vec ? half / 4 : half) + 255) / 256;
+  if (blocks > sm_count() * 16) blocks = sm_count() * 16;
+  const unsigned grid = static_cast<unsigned>(blocks);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const float2* tab = reinterpret_cast<const float2*>(rope_table);
+  if (vec) rotate_tail_kernel<bf16, 4><<<grid, 256, 0, st>>>(static_cast<bf16*>(x), ldx, positions, tab, max_pos, n, heads, dim, rot_dim, half);
+  else if (dtype == NVLLM_BF16) rotate_tail_kernel<bf16, 1><<<grid, 256, 0, st>>>(static_cast<bf16*>(x), ldx, positions, tab, max_pos, n, heads, dim, rot_dim, half);
+  else rotate_tail_kernel<float, 1><<<grid, 256, 0, st>>>(static_cast<float*>(x), ldx, positions, tab, max_pos, n, heads, dim, rot_dim, half);
+  NVLLM_LAUNCH_CHECK("rotate_tail_kernel");
   return 0;
 }
 

@@ -19,6 +19,8 @@ struct LinArgs {
   int64_t up_off;             // GLU: element offset of the `up` rows relative to the `gate` rows inside w
   float limit;                // GLU clamp
   int act;                    // epilogue of the plain product: 0 none, 2 relu(v)^2
+  const float* row_scale;     // factor on row m of x, applied to the accumulators (the product is linear in it)
+  const float* gate; int64_t ldg, bsg;   // y *= sigmoid(gate[m * ldg + b * bsg + n])
 };
 
 template <typename T> __device__ __forceinline__ float ldf(const T* p);
@@ -92,14 +94,15 @@ __global__ void __launch_bounds__(256) linear_tile_kernel(const LinArgs a) {
   for (int i = 0; i < 2; ++i) {
     const int m = m0 + ty * 2 + i;
     if (m >= a.M || (a.row_src && a.row_src[m] < 0)) continue;
+    const float rs = a.row_scale ? a.row_scale[m] : 1.0f;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx + 16 * j;
       if (n >= a.N) continue;
-      float v = acc[i][j];
+      float v = acc[i][j] * rs;
       if (GLU) {
         // bf16 models round gate and up to bf16 before the activation, as a separate projection would have
-        float g = v, u = acu[i][j];
+        float g = v, u = acu[i][j] * rs;
         if (sizeof(TI) == 2) { g = __bfloat162float(__float2bfloat16_rn(g)); u = __bfloat162float(__float2bfloat16_rn(u)); }
         v = a.act == 3 ? g / (1.0f + expf(-g)) * u : glu_clamped(g, u, a.limit);
       } else if (a.act == 2) {
@@ -107,6 +110,7 @@ __global__ void __launch_bounds__(256) linear_tile_kernel(const LinArgs a) {
         v = fmaxf(v, 0.f);
         v *= v;
       }
+      if (a.gate) v *= 1.0f / (1.0f + expf(-a.gate[static_cast<int64_t>(m) * a.ldg + b * a.bsg + n]));
       stf(y + static_cast<int64_t>(m) * a.ldy + n, v);
     }
   }
@@ -152,6 +156,7 @@ __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + lo
 // kind 0: out[i, c] = silu(in[i, c]) * in[i, ff + c] (in: [n, 2 ff]);  kind 1: out[i, c] = relu(in[i, c])^2 (in: [n, ff]);
 // kind 2: out[i, c] = xielu(in[i, c]) with the two learned numbers params[0..1] (in: [n, ff]):
 //         z > 0: softplus(p0) z^2 + z / 2;   z <= 0: (1/2 + softplus(p1)) (exp(z) - 1 - z) + z / 2
+// kind 3: out[i, c] = gelu_tanh(in[i, c]) * in[i, ff + c] (in: [n, 2 ff])
 template <typename T>
 __global__ void ff_activation_kernel(T* __restrict__ out, const T* __restrict__ in, int64_t n, int ff, int kind, const float* __restrict__ params) {
   const int64_t total = n * ff;
@@ -160,9 +165,9 @@ __global__ void ff_activation_kernel(T* __restrict__ out, const T* __restrict__ 
        i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
     const int64_t r = i / ff, c = i - r * ff;
     float v;
-    if (kind == 0) {
+    if (kind == 0 || kind == 3) {
       const float g = ldf(in + r * 2 * ff + c);
-      v = g / (1.0f + expf(-g)) * ldf(in + r * 2 * ff + ff + c);
+      v = (kind == 3 ? gelu_tanh(g) : g / (1.0f + expf(-g))) * ldf(in + r * 2 * ff + ff + c);
     } else if (kind == 2) {
       const float z = ldf(in + i);
       v = z > 0.f ? fmaf(ap * z, z, 0.5f * z) : fmaf(an, expm1f(z) - z, 0.5f * z);
@@ -182,13 +187,13 @@ __global__ void __launch_bounds__(256) ff_activation_vec8_kernel(bf16* __restric
   for (int64_t i = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; i < total;
        i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
     float a[8], o[8];
-    if (kind == 0) {
+    if (kind == 0 || kind == 3) {
       const int64_t r = i / ff8, c = i - r * ff8;
       float u[8];
       unpack8(ld_nc_16(reinterpret_cast<const uint4*>(in) + r * 2 * ff8 + c), a);
       unpack8(ld_nc_16(reinterpret_cast<const uint4*>(in) + r * 2 * ff8 + ff8 + c), u);
 #pragma unroll
-      for (int j = 0; j < 8; ++j) o[j] = a[j] / (1.0f + expf(-a[j])) * u[j];
+      for (int j = 0; j < 8; ++j) o[j] = (kind == 3 ? gelu_tanh_fast(a[j]) : a[j] / (1.0f + expf(-a[j]))) * u[j];
     } else {
       unpack8(ld_nc_16(reinterpret_cast<const uint4*>(in) + i), a);
 #pragma unroll
@@ -197,6 +202,62 @@ __global__ void __launch_bounds__(256) ff_activation_vec8_kernel(bf16* __restric
         else { const float v = fmaxf(a[j], 0.f); o[j] = v * v; }
       }
     }
+    reinterpret_cast<uint4*>(out)[i] = pack8(o);
+  }
+}
+
+// y *= sigmoid(gate), element by element, in place (y in the operand type, gate f32): VEC values per access.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) sigmoid_gate_kernel(T* __restrict__ y, int64_t ldy, const float* __restrict__ gate, int64_t ldg, int64_t n, int cols) {
+  const int64_t total = n * (cols / VEC);
+  for (int64_t i = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; i < total; i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
+    const int64_t r = i / (cols / VEC);
+    const int c = static_cast<int>(i - r * (cols / VEC)) * VEC;
+    T* p = y + r * ldy + c;
+    const float* g = gate + r * ldg + c;
+    if (VEC == 8) {   // T is bf16 here
+      float v[8];
+      unpack8(*reinterpret_cast<const uint4*>(p), v);
+      const float4 g0 = reinterpret_cast<const float4*>(g)[0], g1 = reinterpret_cast<const float4*>(g)[1];
+      const float gg[8] = {g0.x, g0.y, g0.z, g0.w, g1.x, g1.y, g1.z, g1.w};
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[j] *= 1.0f / (1.0f + expf(-gg[j]));
+      *reinterpret_cast<uint4*>(p) = pack8(v);
+    } else {
+      stf(p, ldf(p) * (1.0f / (1.0f + expf(-*g))));
+    }
+  }
+}
+
+// A token's own row of a side table, gated: out[t, c] = gelu_tanh(gate[t, c]) * table[ids[t], col0 + c], gate f32.
+template <typename T>
+__global__ void __launch_bounds__(256) token_gate_kernel(T* __restrict__ out, const float* __restrict__ gate, int64_t ldg, const T* __restrict__ table,
+                                                         int64_t ld_table, int64_t col0, const int64_t* __restrict__ ids, int vocab, int64_t n, int dim) {
+  const int64_t total = n * dim;
+  for (int64_t i = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; i < total; i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
+    const int64_t t = i / dim;
+    const int c = static_cast<int>(i - t * dim);
+    int64_t id = ids[t];
+    id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
+    stf(out + i, gelu_tanh(gate[t * ldg + c]) * ldf(table + id * ld_table + col0 + c));
+  }
+}
+// The same with 16-byte accesses (bf16; dim, ld_table, col0 multiples of 8, ldg of 4).
+__global__ void __launch_bounds__(256) token_gate_vec8_kernel(bf16* __restrict__ out, const float* __restrict__ gate, int64_t ldg,
+                                                              const bf16* __restrict__ table, int64_t ld_table, int64_t col0,
+                                                              const int64_t* __restrict__ ids, int vocab, int64_t n, int dim8) {
+  const int64_t total = n * dim8;
+  for (int64_t i = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; i < total; i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
+    const int64_t t = i / dim8;
+    const int c = static_cast<int>(i - t * dim8) * 8;
+    int64_t id = ids[t];
+    id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
+    float e[8], o[8];
+    unpack8(ld_nc_16(reinterpret_cast<const uint4*>(table + id * ld_table + col0 + c)), e);
+    const float4 g0 = *reinterpret_cast<const float4*>(gate + t * ldg + c), g1 = *reinterpret_cast<const float4*>(gate + t * ldg + c + 4);
+    const float gg[8] = {g0.x, g0.y, g0.z, g0.w, g1.x, g1.y, g1.z, g1.w};
+#pragma unroll
+    for (int j = 0; j < 8; ++j) o[j] = gelu_tanh_fast(gg[j]) * e[j];
     reinterpret_cast<uint4*>(out)[i] = pack8(o);
   }
 }
@@ -262,7 +323,10 @@ __global__ void __launch_bounds__(128) linear_mma_kernel(const LinArgs a) {
 #pragma unroll
       for (int c = 0; c < 2; ++c) {
         const int n = n0 + nt * 8 + 2 * tq4 + c;
-        if (n < a.N) stf(y + static_cast<int64_t>(m) * a.ldy + n, acc[nt][2 * i + c]);
+        if (n >= a.N) continue;
+        float v = acc[nt][2 * i + c];
+        if (a.gate) v *= 1.0f / (1.0f + expf(-a.gate[static_cast<int64_t>(m) * a.ldg + b * a.bsg + n]));
+        stf(y + static_cast<int64_t>(m) * a.ldy + n, v);
       }
   }
 }
@@ -306,17 +370,24 @@ using namespace nvllm;
 extern "C" int nvllm_linear(void* y, const void* x, const void* w, int32_t m, int32_t n, int32_t k, int64_t ldx, int64_t ldw,
                             int64_t ldy, int32_t batch, int64_t bsx, int64_t bsw, int64_t bsy, int32_t dtype,
                             int32_t out_dtype, void* stream) {
+  return nvllm_linear_gated(y, x, w, m, n, k, ldx, ldw, ldy, batch, bsx, bsw, bsy, nullptr, 0, 0, dtype, out_dtype, stream);
+}
+
+extern "C" int nvllm_linear_gated(void* y, const void* x, const void* w, int32_t m, int32_t n, int32_t k, int64_t ldx, int64_t ldw,
+                                  int64_t ldy, int32_t batch, int64_t bsx, int64_t bsw, int64_t bsy, const float* gate, int64_t ldg,
+                                  int64_t bsg, int32_t dtype, int32_t out_dtype, void* stream) {
   NVLLM_CHECK_ARG(m >= 0 && n > 0 && k > 0 && batch > 0, NVLLM_ERR_ARG, "linear: m=%d n=%d k=%d batch=%d", m, n, k, batch);
   NVLLM_CHECK_ARG(ldx >= k && ldw >= k && ldy >= n, NVLLM_ERR_ARG, "linear: leading dimensions");
   NVLLM_CHECK_ARG((dtype == NVLLM_BF16 || dtype == NVLLM_F32) && (out_dtype == NVLLM_BF16 || out_dtype == NVLLM_F32),
                   NVLLM_ERR_DTYPE, "linear: dtype %d / %d", dtype, out_dtype);
   if (m == 0) return 0;
   NVLLM_CHECK_ARG(y && x && w, NVLLM_ERR_ARG, "linear: NULL");
+  NVLLM_CHECK_ARG(gate == nullptr || ldg >= n, NVLLM_ERR_ARG, "linear: gate rows %lld apart, %d columns", (long long)ldg, n);
   // dense bf16 problems that fit the tensor-core kernel's rules go there
-  if (dtype == NVLLM_BF16 && batch == 1 && k % 64 == 0 && n % 8 == 0 && ldx % 8 == 0 && ldw % 8 == 0 && ldy % 8 == 0 &&
+  if (dtype == NVLLM_BF16 && gate == nullptr && batch == 1 && k % 64 == 0 && n % 8 == 0 && ldx % 8 == 0 && ldw % 8 == 0 && ldy % 8 == 0 &&
       aligned16(y) && aligned16(x) && aligned16(w))
     return nvllm_gemm_bf16(y, x, w, m, n, k, ldx, ldw, ldy, out_dtype, nullptr, 0, stream);
-  LinArgs a{y, x, w, m, n, k, ldx, ldw, ldy, bsx, bsw, bsy, nullptr, nullptr, 0, 0.f, 0};
+  LinArgs a{y, x, w, m, n, k, ldx, ldw, ldy, bsx, bsw, bsy, nullptr, nullptr, 0, 0.f, 0, nullptr, gate, ldg, bsg};
   // other bf16 problems with 16-byte rows (per-head batches, reduction sizes that are not multiples of 64): mma.sync tiles
   if (dtype == NVLLM_BF16 && knobs().linear_mma && mma_applies(a)) return launch_mma(a, batch, out_dtype, static_cast<cudaStream_t>(stream));
   return launch_tile<false>(a, (m + BM - 1) / BM, batch, dtype, out_dtype, static_cast<cudaStream_t>(stream));
@@ -326,6 +397,14 @@ extern "C" int nvllm_linear_grouped(void* y, const void* x, const void* w, int32
                                     int64_t ldx, int64_t ldw, int64_t ldy, int64_t group_stride_w, const int32_t* row_src,
                                     const int32_t* tile_group, int32_t glu, float limit, int32_t dtype, int32_t out_dtype,
                                     void* stream) {
+  return nvllm_linear_grouped_scaled(y, x, w, max_rows, n, k, ldx, ldw, ldy, group_stride_w, row_src, nullptr, tile_group, glu, limit, dtype, out_dtype,
+                                     stream);
+}
+
+extern "C" int nvllm_linear_grouped_scaled(void* y, const void* x, const void* w, int32_t max_rows, int32_t n, int32_t k,
+                                           int64_t ldx, int64_t ldw, int64_t ldy, int64_t group_stride_w, const int32_t* row_src,
+                                           const float* row_scale, const int32_t* tile_group, int32_t glu, float limit, int32_t dtype,
+                                           int32_t out_dtype, void* stream) {
   NVLLM_CHECK_ARG(max_rows >= 0 && n > 0 && k > 0 && max_rows % BM == 0, NVLLM_ERR_ARG,
                   "linear_grouped: max_rows=%d (multiple of 32) n=%d k=%d", max_rows, n, k);
   NVLLM_CHECK_ARG((dtype == NVLLM_BF16 || dtype == NVLLM_F32) && (out_dtype == NVLLM_BF16 || out_dtype == NVLLM_F32),
@@ -334,7 +413,7 @@ extern "C" int nvllm_linear_grouped(void* y, const void* x, const void* w, int32
   NVLLM_CHECK_ARG(y && x && w, NVLLM_ERR_ARG, "linear_grouped: NULL");
   // GLU: every group's weight block is [gate rows (n) | up rows (n)] x k
   LinArgs a{y, x, w, max_rows, n, k, ldx, ldw, ldy, 0, group_stride_w, 0, row_src, tile_group,
-            static_cast<int64_t>(n) * ldw, limit, glu == 2 ? 2 : (glu == 3 ? 3 : 0)};
+            static_cast<int64_t>(n) * ldw, limit, glu == 2 ? 2 : (glu == 3 ? 3 : 0), row_scale, nullptr, 0, 0};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   return (glu == 1 || glu == 3) ? launch_tile<true>(a, max_rows / BM, 1, dtype, out_dtype, st)
              : launch_tile<false>(a, max_rows / BM, 1, dtype, out_dtype, st);
@@ -369,7 +448,7 @@ extern "C" int nvllm_ff_activation(void* out, const void* in, int32_t n, int32_t
 
 extern "C" int nvllm_ff_activation_params(void* out, const void* in, int32_t n, int32_t ff, int32_t kind, const float* params, int32_t dtype,
                                           void* stream) {
-  NVLLM_CHECK_ARG(n >= 0 && ff > 0 && kind >= 0 && kind <= 2 && (kind != 2 || params != nullptr), NVLLM_ERR_ARG,
+  NVLLM_CHECK_ARG(n >= 0 && ff > 0 && kind >= 0 && kind <= 3 && (kind != 2 || params != nullptr), NVLLM_ERR_ARG,
                   "ff_activation: n=%d ff=%d kind=%d (kind 2 needs its two parameters)", n, ff, kind);
   NVLLM_CHECK_ARG(dtype == NVLLM_BF16 || dtype == NVLLM_F32, NVLLM_ERR_DTYPE, "ff_activation: dtype %d", dtype);
   if (n == 0) return 0;
@@ -388,5 +467,44 @@ extern "C" int nvllm_ff_activation_params(void* out, const void* in, int32_t n, 
   if (dtype == NVLLM_BF16) ff_activation_kernel<bf16><<<static_cast<unsigned>(blocks), 256, 0, st>>>(static_cast<bf16*>(out), static_cast<const bf16*>(in), n, ff, kind, params);
   else ff_activation_kernel<float><<<static_cast<unsigned>(blocks), 256, 0, st>>>(static_cast<float*>(out), static_cast<const float*>(in), n, ff, kind, params);
   NVLLM_LAUNCH_CHECK("ff_activation_kernel");
+  return 0;
+}
+
+extern "C" int nvllm_sigmoid_gate(void* y, int64_t ldy, const float* gate, int64_t ldg, int32_t n, int32_t cols, int32_t dtype, void* stream) {
+  NVLLM_CHECK_ARG(n >= 0 && cols > 0 && ldy >= cols && ldg >= cols, NVLLM_ERR_ARG, "sigmoid_gate: n=%d cols=%d", n, cols);
+  NVLLM_CHECK_ARG(dtype == NVLLM_BF16 || dtype == NVLLM_F32, NVLLM_ERR_DTYPE, "sigmoid_gate: dtype %d", dtype);
+  if (n == 0) return 0;
+  NVLLM_CHECK_ARG(y && gate, NVLLM_ERR_ARG, "sigmoid_gate: NULL");
+  const bool vec = dtype == NVLLM_BF16 && cols % 8 == 0 && ldy % 8 == 0 && ldg % 4 == 0 && aligned16(y) && aligned16(gate);
+  int64_t blocks = (static_cast<int64_t>(n) * (vec ? cols / 8 : cols) + 255) / 256;
+  if (blocks > sm_count() * 16) blocks = sm_count() * 16;
+  const unsigned grid = static_cast<unsigned>(blocks);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (vec) sigmoid_gate_kernel<bf16, 8><<<grid, 256, 0, st>>>(static_cast<bf16*>(y), ldy, gate, ldg, n, cols);
+  else if (dtype == NVLLM_BF16) sigmoid_gate_kernel<bf16, 1><<<grid, 256, 0, st>>>(static_cast<bf16*>(y), ldy, gate, ldg, n, cols);
+  else sigmoid_gate_kernel<float, 1><<<grid, 256, 0, st>>>(static_cast<float*>(y), ldy, gate, ldg, n, cols);
+  NVLLM_LAUNCH_CHECK("sigmoid_gate_kernel");
+  return 0;
+}
+
+extern "C" int nvllm_token_gate(void* out, const float* gate, int64_t ldg, const void* table, int64_t ld_table, int64_t col0, const int64_t* ids,
+                                int32_t vocab, int32_t n, int32_t dim, int32_t dtype, void* stream) {
+  NVLLM_CHECK_ARG(n >= 0 && dim > 0 && vocab > 0 && ldg >= dim && col0 >= 0 && ld_table >= col0 + dim, NVLLM_ERR_ARG,
+                  "token_gate: n=%d dim=%d, columns %lld.. of rows of %lld", n, dim, (long long)col0, (long long)ld_table);
+  NVLLM_CHECK_ARG(dtype == NVLLM_BF16 || dtype == NVLLM_F32, NVLLM_ERR_DTYPE, "token_gate: dtype %d", dtype);
+  if (n == 0) return 0;
+  NVLLM_CHECK_ARG(out && gate && table && ids, NVLLM_ERR_ARG, "token_gate: NULL");
+  const bool vec = dtype == NVLLM_BF16 && dim % 8 == 0 && ld_table % 8 == 0 && col0 % 8 == 0 && ldg % 4 == 0 && aligned16(out) && aligned16(gate) && aligned16(table);
+  int64_t blocks = (static_cast<int64_t>(n) * (vec ? dim / 8 : dim) + 255) / 256;
+  if (blocks > sm_count() * 16) blocks = sm_count() * 16;
+  const unsigned grid = static_cast<unsigned>(blocks);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (vec)
+    token_gate_vec8_kernel<<<grid, 256, 0, st>>>(static_cast<bf16*>(out), gate, ldg, static_cast<const bf16*>(table), ld_table, col0, ids, vocab, n, dim / 8);
+  else if (dtype == NVLLM_BF16)
+    token_gate_kernel<bf16><<<grid, 256, 0, st>>>(static_cast<bf16*>(out), gate, ldg, static_cast<const bf16*>(table), ld_table, col0, ids, vocab, n, dim);
+  else
+    token_gate_kernel<float><<<grid, 256, 0, st>>>(static_cast<float*>(out), gate, ldg, static_cast<const float*>(table), ld_table, col0, ids, vocab, n, dim);
+  NVLLM_LAUNCH_CHECK("token_gate_kernel");
   return 0;
 }

@@ -6,6 +6,7 @@
 //
 //   s = softmax(z) over all router outputs (real experts first, then identity experts)
 //   chosen = the `top` largest of s + bias (ties: lowest index);  w_k = s[chosen_k] / (sum_k s[chosen_k] + 1e-20) * scale
+//   (nvllm_moe_route_logits, nvllm_moe_route_sigmoid: choice and weights from the logits in other ways)
 //   out[t] = sum_k w_k * (chosen_k < experts ? expert_out[row of (t, k)] : x[t]) + shared[t]
 #include "common.cuh"
 
@@ -111,19 +112,60 @@ __global__ void __launch_bounds__(128) moe_route_logits_kernel(int32_t* __restri
   }
 }
 
+// Routing on sigmoid scores: the `top` largest of logits + bias (the sigmoid keeps their order; ties: lowest index); the weights
+// are the chosen experts' scores sigmoid(logits + bias) as they are.  One warp per token.
+__global__ void __launch_bounds__(128) moe_route_sigmoid_kernel(int32_t* __restrict__ idx, float* __restrict__ wts,
+                                                                const float* __restrict__ logits, const float* __restrict__ bias,
+                                                                int64_t ld, int n, int e_total, int top) {
+  extern __shared__ float sm[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t = blockIdx.x * 4 + warp;
+  if (t >= n) return;
+  float* c = sm + static_cast<size_t>(warp) * e_total;
+  const float* z = logits + static_cast<int64_t>(t) * ld;
+  for (int e = lane; e < e_total; e += 32) c[e] = z[e] + (bias ? bias[e] : 0.f);
+  __syncwarp();
+  for (int k = 0; k < top; ++k) {
+    float best = -INFINITY;
+    int bi = 0x7fffffff;
+    for (int e = lane; e < e_total; e += 32) {
+      const float v = c[e];
+      if (v > best) { best = v; bi = e; }   // ascending e per lane: the first maximum wins
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+      if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
+    }
+    if (bi == 0x7fffffff) bi = 0;  // every logit NaN / -inf: degenerate, keep indices valid
+    if (lane == 0) {
+      idx[static_cast<int64_t>(t) * top + k] = bi;
+      wts[static_cast<int64_t>(t) * top + k] = 1.0f / (1.0f + expf(-best));
+      c[bi] = -INFINITY;
+    }
+    __syncwarp();
+  }
+}
+
 // Counting sort of the assignments by expert, one CTA.  Output layout: expert e owns rows [off[e], off[e] + cnt[e]) of the
 // grouped buffers, off[e] a multiple of the tile height so that no tile spans two experts.
 //   row_token[r]  token whose activations row r reads (-1: padding)
 //   tile_expert[i] expert of tile i (-1: unused tile)
 //   slot_row[t*top + k] row of assignment (t, k), or -1 when it chose an identity expert
+//   row_weight[r] (nullable) the assignment's weight wts[t*top + k] beside its row (0: padding), for experts that scale their input
 __global__ void __launch_bounds__(1024) moe_sort_kernel(int32_t* __restrict__ row_token, int32_t* __restrict__ tile_expert,
-                                                        int32_t* __restrict__ slot_row, const int32_t* __restrict__ idx,
+                                                        int32_t* __restrict__ slot_row, float* __restrict__ row_weight,
+                                                        const int32_t* __restrict__ idx, const float* __restrict__ wts,
                                                         int n_assign, int top, int experts, int max_rows, int tile) {
   extern __shared__ int32_t sh[];
   int32_t* cnt = sh;             // [experts]
   int32_t* off = sh + experts;   // [experts + 1]
   for (int e = threadIdx.x; e < experts; e += blockDim.x) cnt[e] = 0;
-  for (int r = threadIdx.x; r < max_rows; r += blockDim.x) row_token[r] = -1;
+  for (int r = threadIdx.x; r < max_rows; r += blockDim.x) {
+    row_token[r] = -1;
+    if (row_weight != nullptr) row_weight[r] = 0.f;
+  }
   for (int i = threadIdx.x; i < max_rows / tile; i += blockDim.x) tile_expert[i] = -1;
   __syncthreads();
   for (int a = threadIdx.x; a < n_assign; a += blockDim.x) {
@@ -148,6 +190,7 @@ __global__ void __launch_bounds__(1024) moe_sort_kernel(int32_t* __restrict__ ro
       const int r = off[e] + slot_row[a];
       slot_row[a] = r;
       row_token[r] = a / top;
+      if (row_weight != nullptr) row_weight[r] = wts[a];
     }
   }
 }
@@ -167,7 +210,7 @@ __global__ void moe_combine_kernel(T* __restrict__ out, const T* __restrict__ ex
       const int64_t a = t * top + k;
       const int r = slot_row[a];
       const float v = r >= 0 ? ldf(expert_out + static_cast<int64_t>(r) * hidden + c) : ldf(x + i);
-      acc = fmaf(wts[a], v, acc);
+      acc = fmaf(wts ? wts[a] : 1.0f, v, acc);
     }
     if (shared_out) acc += ldf(shared_out + i);
     stf(out + i, acc);
@@ -196,7 +239,7 @@ __global__ void moe_combine_vec8_kernel(bf16* __restrict__ out, const bf16* __re
       const int64_t a = t * top + k;
       const int r = slot_row[a];
       unpack8(r >= 0 ? reinterpret_cast<const uint4*>(expert_out)[static_cast<int64_t>(r) * hidden8 + c] : reinterpret_cast<const uint4*>(x)[i], v);
-      const float w = wts[a];
+      const float w = wts ? wts[a] : 1.0f;
 #pragma unroll
       for (int j = 0; j < 8; ++j) acc[j] = fmaf(w, v[j], acc[j]);
     }
@@ -263,6 +306,18 @@ extern "C" int nvllm_moe_route_logits(int32_t* topk_idx, float* topk_w, const fl
   return 0;
 }
 
+extern "C" int nvllm_moe_route_sigmoid(int32_t* topk_idx, float* topk_w, const float* logits, int64_t ld, const float* bias, int32_t n,
+                                       int32_t experts, int32_t top, void* stream) {
+  NVLLM_CHECK_ARG(n >= 0 && experts > 0 && top > 0 && top <= experts && experts <= 3072 && ld >= experts, NVLLM_ERR_ARG,
+                  "moe_route_sigmoid: n=%d experts=%d top=%d", n, experts, top);
+  if (n == 0) return 0;
+  NVLLM_CHECK_ARG(topk_idx && topk_w && logits, NVLLM_ERR_ARG, "moe_route_sigmoid: NULL");
+  const size_t smem = static_cast<size_t>(4) * experts * sizeof(float);
+  moe_route_sigmoid_kernel<<<(n + 3) / 4, 128, smem, static_cast<cudaStream_t>(stream)>>>(topk_idx, topk_w, logits, bias, ld, n, experts, top);
+  NVLLM_LAUNCH_CHECK("moe_route_sigmoid_kernel");
+  return 0;
+}
+
 extern "C" int32_t nvllm_moe_max_rows(int32_t n_tokens, int32_t top, int32_t experts, int32_t tile_rows) {
   if (tile_rows <= 0) return 0;
   const int64_t a = static_cast<int64_t>(n_tokens) * top + static_cast<int64_t>(experts) * (tile_rows - 1);
@@ -271,13 +326,20 @@ extern "C" int32_t nvllm_moe_max_rows(int32_t n_tokens, int32_t top, int32_t exp
 
 extern "C" int nvllm_moe_sort(int32_t* row_token, int32_t* tile_expert, int32_t* slot_row, const int32_t* topk_idx,
                               int32_t n, int32_t top, int32_t experts, int32_t max_rows, int32_t tile_rows, void* stream) {
+  return nvllm_moe_sort_weighted(row_token, nullptr, tile_expert, slot_row, topk_idx, nullptr, n, top, experts, max_rows, tile_rows, stream);
+}
+
+extern "C" int nvllm_moe_sort_weighted(int32_t* row_token, float* row_weight, int32_t* tile_expert, int32_t* slot_row, const int32_t* topk_idx,
+                                       const float* topk_w, int32_t n, int32_t top, int32_t experts, int32_t max_rows, int32_t tile_rows,
+                                       void* stream) {
+  NVLLM_CHECK_ARG(row_weight == nullptr || topk_w != nullptr, NVLLM_ERR_ARG, "moe_sort: weights per row without weights per assignment");
   NVLLM_CHECK_ARG(n >= 0 && top > 0 && experts >= 0 && experts <= 8192 && (tile_rows == 32 || tile_rows == 128) &&
                       max_rows % tile_rows == 0 && max_rows >= nvllm_moe_max_rows(n, top, experts, tile_rows), NVLLM_ERR_ARG,
                   "moe_sort: n=%d top=%d experts=%d max_rows=%d tile_rows=%d", n, top, experts, max_rows, tile_rows);
   if (n == 0) return 0;
   NVLLM_CHECK_ARG(row_token && tile_expert && slot_row && topk_idx, NVLLM_ERR_ARG, "moe_sort: NULL");
   const size_t smem = (2 * static_cast<size_t>(experts) + 1) * sizeof(int32_t);
-  moe_sort_kernel<<<1, 1024, smem, static_cast<cudaStream_t>(stream)>>>(row_token, tile_expert, slot_row, topk_idx, n * top, top,
+  moe_sort_kernel<<<1, 1024, smem, static_cast<cudaStream_t>(stream)>>>(row_token, tile_expert, slot_row, row_weight, topk_idx, topk_w, n * top, top,
                                                                       experts, max_rows, tile_rows);
   NVLLM_LAUNCH_CHECK("moe_sort_kernel");
   return 0;
@@ -289,7 +351,7 @@ extern "C" int nvllm_moe_combine(void* out, const void* expert_out, const void* 
   NVLLM_CHECK_ARG(n >= 0 && hidden > 0 && top > 0, NVLLM_ERR_ARG, "moe_combine: sizes");
   NVLLM_CHECK_ARG(dtype == NVLLM_BF16 || dtype == NVLLM_F32, NVLLM_ERR_DTYPE, "moe_combine: dtype %d", dtype);
   if (n == 0) return 0;
-  NVLLM_CHECK_ARG(out && x && topk_idx && topk_w && slot_row && (expert_out || experts == 0), NVLLM_ERR_ARG, "moe_combine: NULL");
+  NVLLM_CHECK_ARG(out && x && topk_idx && slot_row && (expert_out || experts == 0), NVLLM_ERR_ARG, "moe_combine: NULL");
   const int64_t total = static_cast<int64_t>(n) * hidden;
   int64_t blocks = (total + 255) / 256;
   if (blocks > sm_count() * 16) blocks = sm_count() * 16;
