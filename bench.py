@@ -53,7 +53,7 @@ def parse():
     ap.add_argument("--warmup", type=int, default=4)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--model", default=None, help="override the workload model (qwen3-0.6b | qwen3-8b | qwen3-32b)")
-    ap.add_argument("--workload", default="decode", choices=["decode", "prefix", "kosazen", "talapel", "zudatar", "zasorax", "kalesun"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "prefix", "kosazen", "talapel", "zudatar", "zasorax", "kalesun", "fomerax"],
                     help="kosazen: prefill / decode throughput and a per-kernel roofline table of the Kosazen architecture "
                          "(latent attention + mixture of experts) beside Qwen3 models of equal layer sizes, random weights; "
                          "talapel: the same for the Talapel architecture (capped attention beside a state-space mixer, retention, "
@@ -61,7 +61,9 @@ def parse():
                          "attention in a window, gated delta rule); zasorax: the same for the Zasorax architecture (post-norm blocks, "
                          "chunked attention with a distance bias, rotated values, experts routed on logits); kalesun: the Kalesun architecture "
                          "(norm after the sum, windowed attention with kept first keys, gated delta rule, gated linear attention) beside "
-                         "Zudatar and Zasorax models of equal layer sizes")
+                         "Zudatar and Zasorax models of equal layer sizes; fomerax: the Fomerax architecture (capped attention with a slope "
+                         "per head, latent attention with a rotated key part, experts that scale their input, token inputs) beside "
+                         "Zudatar, Talapel and Kalesun models of equal layer sizes")
     ap.add_argument("--seqs", type=int, default=None)
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-parity", action="store_true", help="skip the in-run parity checks (profiling runs)")
@@ -824,6 +826,32 @@ def kalesun_config(z):
             "layers": [kinds[i % 4] for i in range(z["layers"])]}
 
 
+# Fomerax: a capped attention layer with a dense feed-forward, a latent layer with experts, a capped attention layer with experts and
+# a latent layer with a dense feed-forward, a token input behind each; the sizes (width, heads, window, ranks, feed-forward,
+# experts) are those of the Zudatar, Talapel and Kalesun arms it is measured beside: latent attention, sandwich norms and dense
+# layers have their like kernels in the first, capped attention in the second, experts in the third.
+FOMERAX_SIZES = {
+    "w2048": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=128, rot_dim=64, window=512, kv_rank=512, q_rank=768, dense_ff=8192, ff=1024, experts=32,
+                  top=4, side=256, layers=4, vocab=32768),
+    "w4096": dict(width=4096, heads=32, kv_heads=8, dim=128, vdim=128, rot_dim=64, window=512, kv_rank=512, q_rank=1536, dense_ff=12288, ff=1536, experts=32,
+                  top=4, side=256, layers=4, vocab=32768),
+}
+
+
+def fomerax_config(z):
+    dense = {"kind": "dense", "ff": z["dense_ff"]}
+    moe = {"kind": "moe", "expert": {"ff": z["ff"]}, "router": {"experts": z["experts"], "top": z["top"]}}
+    att = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["vdim"], "scale": z["dim"] ** -0.5, "softcap": 50.0,
+           "q_temp": {"coef": 0.1, "every": 256}}
+    lat = {"heads": z["heads"], "dim": z["dim"], "rot_dim": z["rot_dim"], "vdim": z["vdim"], "q_rank": z["q_rank"], "kv_rank": z["kv_rank"],
+           "scale": (z["dim"] + z["rot_dim"]) ** -0.5, "mask": {"size": z["window"]},
+           "rot": {"base": 10000.0, "dims": z["rot_dim"], "scaling": {"factor": 8.0, "fast": 32.0, "slow": 1.0, "original": 4096}}}
+    kinds = [{"type": "attention", "mixer": att, "mlp": dense}, {"type": "latent_attention", "mixer": lat, "mlp": moe},
+             {"type": "attention", "mixer": att, "mlp": moe}, {"type": "latent_attention", "mixer": lat, "mlp": dense}]
+    return {"architecture": "Fomerax", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5}, "token_side": {"dim": z["side"]},
+            "layers": [kinds[i % 4] for i in range(z["layers"])]}
+
+
 def kernel_rooflines(z, arch, n_tok, ctx, decode, hbm, tf):
     """Algorithmic work of the named launches of ONE layer at n_tok tokens (context ctx per sequence): {name: (flop, bytes)}."""
     W, H, L = z["width"], z["heads"], ctx
@@ -922,6 +950,39 @@ def kernel_rooflines(z, arch, n_tok, ctx, decode, hbm, tf):
         f32_tf = 148 * 128 * 2 * 1.965e9 / 1e12   # everything that enters a recurrence is f32 by definition of the design
         f32_names = ("head_delta_recurrence", "channel_recurrence", "low_rank_decay", "causal_conv")
         return {k: max(f / ((f32_tf if k in f32_names else tf) * 1e12), b / (hbm * 1e9)) * 1e6 for k, (f, b) in out.items()}
+    if arch == "fomerax":
+        D, V, G, rd, R, QR, w, sd = z["dim"], z["vdim"], z["kv_heads"], z["rot_dim"], z["kv_rank"], z["q_rank"], z["window"], z["side"]
+        seqs = n_tok if decode else max(1, n_tok // L)
+        wpairs = n_tok * min(w, L) if decode else seqs * (min(w, L) * (min(w, L) + 1) / 2 + max(0, L - w) * w)
+        keys_read = n_tok * min(w, L) if decode else n_tok
+        gemm = lambda n, k, out=4: (2 * n_tok * n * k, 2 * n * k + n_tok * (2 * k + out * n))
+        qkv = H * D + G * D + G * V
+        out["attention q k v g projection"] = gemm(qkv + H * V, W)
+        out["attn_store"] = (0, n_tok * qkv * 6)
+        # (all causal pairs, as if every head looked at every key)
+        out["sloped_attention"] = (2 * pairs * H * (D + V), (n_tok * L if decode else n_tok) * G * (D + V) * 2 + n_tok * H * (D + 3 * V) * 2)
+        out["latent dq dkv g projection"] = gemm(QR + R + rd + H * V, W)
+        out["latent_norm_store"] = (0, n_tok * (QR + R + rd) * 6)
+        out["query up-projection"] = gemm(H * (D + rd), QR, 2)
+        out["rotate_tail (queries)"] = (0, n_tok * H * rd * 4)
+        out["q absorb (per-head GEMMs)"] = out["q absorb (per-head linear)"] = (2 * n_tok * H * D * R, 2 * H * D * R + n_tok * H * (2 * D + 4 * R))
+        out["latent_window_attention"] = (2 * wpairs * H * (2 * R + rd), keys_read * (R + rd) * 2 + n_tok * H * (6 * R + 2 * rd))
+        out["value up-projection + gate (per-head linear)"] = (2 * n_tok * H * V * R, 2 * H * V * R + n_tok * H * (2 * R + 6 * V))
+        out["key / value up-projection"] = gemm(H * (D + V), R, 2)
+        out["window_attention (latent layer, whole prompts)"] = (2 * wpairs * H * (D + rd + V), n_tok * (H * (D + V) + rd) * 2 + n_tok * H * (D + rd + 3 * V) * 2)
+        out["mixer output projection"] = gemm(W, H * V, 2)
+        out["gate / up projection + gelu gate"] = (2 * n_tok * W * 2 * z["dense_ff"], 2 * W * 2 * z["dense_ff"] + n_tok * 2 * (W + z["dense_ff"]))
+        out["down projection"] = (2 * n_tok * W * z["dense_ff"], 2 * W * z["dense_ff"] + n_tok * 2 * (W + z["dense_ff"]))
+        used = min(z["experts"], n_tok * z["top"])
+        out["expert gate / up + silu gate grouped GEMM"] = (2 * n_tok * z["top"] * W * 2 * z["ff"], 2 * used * 2 * z["ff"] * W)
+        out["expert down grouped GEMM"] = (2 * n_tok * z["top"] * W * z["ff"], 2 * used * z["ff"] * W)
+        out["expert row gather"] = (0, n_tok * z["top"] * W * 4)
+        out["moe_combine"] = (0, n_tok * (z["top"] + 1) * W * 2)
+        out["token input gate projection"] = gemm(sd, W)
+        out["token_gate"] = (0, n_tok * sd * 8)
+        out["token input projection"] = gemm(W, sd, 2)
+        out["rms_residual_norm"] = (0, n_tok * W * (4 + 4 + 2 + 2))
+        return {k: max(f / (tf * 1e12), b / (hbm * 1e9)) * 1e6 for k, (f, b) in out.items()}
     if arch == "zudatar":
         D, V, G, R, QR, w = z["dim"], z["vdim"], z["kv_heads"], z["kv_rank"], z["q_rank"], z["window"]
         dH, dG, dD, dV, lr = z["d_heads"], z["d_kv_heads"], z["d_dim"], z["d_vdim"], z["low_rank"]
@@ -989,7 +1050,8 @@ def run_arch_compare(args, new_arch="kosazen", beside=("qwen3",)):
     rng = __import__("numpy").random.default_rng(0)
     result = {"workload": f"{new_arch}-vs-{'-'.join(beside)}", "data": "synthetic", "dtype": "bf16", "prefill": f"{n_prompts} x {plen} tokens per step",
               "decode": f"{dec_b} sequences at context {plen}+", "peaks": {"hbm_gbs": hbm, "bf16_tflops": tf}, "sizes": {}}
-    all_sizes = {"kosazen": ARCH_SIZES, "talapel": TALAPEL_SIZES, "zudatar": ZUDATAR_SIZES, "zasorax": ZASORAX_SIZES, "kalesun": KALESUN_SIZES}
+    all_sizes = {"kosazen": ARCH_SIZES, "talapel": TALAPEL_SIZES, "zudatar": ZUDATAR_SIZES, "zasorax": ZASORAX_SIZES, "kalesun": KALESUN_SIZES,
+                 "fomerax": FOMERAX_SIZES}
     sizes = all_sizes[new_arch]
     only = os.environ.get("BENCH_ARCH_SIZES")          # e.g. "w2048": a subset of the sizes
     for name, z in sizes.items():
@@ -1024,6 +1086,8 @@ def run_arch_compare(args, new_arch="kosazen", beside=("qwen3",)):
                 cfg = E.Config(model_config=zasorax_config(z), **common)
             elif arch == "kalesun":
                 cfg = E.Config(model_config=kalesun_config(z), **common)
+            elif arch == "fomerax":
+                cfg = E.Config(model_config=fomerax_config(z), **common)
             else:
                 cfg = E.Config("qwen3-0.6b", vocab_size=z["vocab"], hidden_size=z["width"], num_hidden_layers=z["layers"],
                                intermediate_size=mlp_q, num_attention_heads=z["heads"],
@@ -1128,6 +1192,10 @@ def main():
     torch.cuda.set_device(local)
     lib = E.lib()
     assert lib.nvllm_device_ok() == 1, "no sm_100 device: the product path has no fallback"
+    if args.workload == "fomerax":
+        assert world == 1, "--workload fomerax is a one-GPU comparison"
+        print(json.dumps(run_arch_compare(args, "fomerax", ("zudatar", "talapel", "kalesun"))), flush=True)
+        return 0
     if args.workload == "kalesun":
         assert world == 1, "--workload kalesun is a one-GPU comparison"
         print(json.dumps(run_arch_compare(args, "kalesun", ("zudatar", "zasorax"))), flush=True)

@@ -619,7 +619,7 @@ __global__ void __launch_bounds__(128) capped_attn_warp_kernel(const AttnArgs a)
 // portion, so a row's result does not depend on how the prompt was cut.  Head sizes are padded to DMAX / VMAX with zeros in
 // shared memory.
 constexpr float kLog2e = 1.4426950408889634f;
-constexpr int kWarps = 8, kRows = 16 * kWarps, kKeys = 64, kThreads = 32 * kWarps;
+constexpr int kWarps = 8, kRows = 16 * kWarps, kKeys = 64;   // (heads beyond 128 values: 16 warps, see launch_mma)
 
 // tanh(x) = 1 - 2 / (2^(2 x log2 e) + 1): two MUFU operations (ex2, rcp), absolute error ~1e-6; exact at both saturations
 // (2^inf -> 1, 2^-inf -> -1).  The one-instruction tanh.approx is 2^-11 relative: too coarse where two scores near the cap
@@ -713,12 +713,13 @@ __device__ __forceinline__ void attn_tile(float (&o)[VMAX / 8][4], float (&m)[2]
   }
 }
 
-template <int DMAX, int VMAX, int EXT>
-__global__ void __launch_bounds__(kThreads, DMAX > 128 ? 1 : 2) capped_attn_mma_kernel(const AttnArgs a, const int32_t* __restrict__ cu_tokens, int n_seqs, int tq,
+template <int DMAX, int VMAX, int EXT, int WARPS>
+__global__ void __launch_bounds__(32 * WARPS, 16 / WARPS) capped_attn_mma_kernel(const AttnArgs a, const int32_t* __restrict__ cu_tokens, int n_seqs, int tq,
                                                               int group) {
+  constexpr int kRows = 16 * WARPS, kThreads = 32 * WARPS;
   constexpr int QS = DMAX + 8, VS = VMAX + 8;       // shared-memory row strides (elements): 16-byte rows, conflict-free ldmatrix
   extern __shared__ __align__(16) unsigned char smem_raw[];
-  bf16* Qs = reinterpret_cast<bf16*>(smem_raw);     // [64][QS]
+  bf16* Qs = reinterpret_cast<bf16*>(smem_raw);     // [kRows][QS]
   bf16* Ks = Qs + kRows * QS;                        // [2][64][QS]
   bf16* Vs = Ks + 2 * kKeys * QS;                    // [2][64][VS]
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gq = lane >> 2, tq4 = lane & 3;
@@ -768,8 +769,9 @@ __global__ void __launch_bounds__(kThreads, DMAX > 128 ? 1 : 2) capped_attn_mma_
     const int32_t blk = table[j / a.block_size];
     return blk >= 0 ? static_cast<int64_t>(blk) * a.block_size + j % a.block_size : -1;
   };
-  // thread -> (key row, every fourth 16-byte chunk of it): no index arithmetic in the copy loop
-  const int lr = tid >> 2, lh = tid & 3;
+  // thread -> (key row, every TPK-th 16-byte chunk of it): no index arithmetic in the copy loop
+  constexpr int TPK = kThreads / kKeys;
+  const int lr = tid / TPK, lh = tid % TPK;
   auto load_tile = [&](int it) {
     const int buf = it & 1;
     bf16* kd = Ks + buf * kKeys * QS + lr * QS;
@@ -778,18 +780,18 @@ __global__ void __launch_bounds__(kThreads, DMAX > 128 ? 1 : 2) capped_attn_mma_
     const bf16* ksrc = slot >= 0 ? kc + slot * a.k_row : kc;
     const bf16* vsrc = slot >= 0 ? vc + slot * a.v_row : vc;
     const int nb = slot >= 0 ? 16 : 0;
-    for (int c = lh; c < och; c += 4) cp_async_16(smem_u32(kd + c * 8), ksrc + (nb ? c * 8 : 0), nb);
+    for (int c = lh; c < och; c += TPK) cp_async_16(smem_u32(kd + c * 8), ksrc + (nb ? c * 8 : 0), nb);
     if (och < dch) {   // the part that all heads share
       const bf16* ssrc = slot >= 0 ? ks + slot * a.ks_row : ks;
-      for (int c = lh; c < dch - och; c += 4) cp_async_16(smem_u32(kd + (och + c) * 8), ssrc + (nb ? c * 8 : 0), nb);
+      for (int c = lh; c < dch - och; c += TPK) cp_async_16(smem_u32(kd + (och + c) * 8), ssrc + (nb ? c * 8 : 0), nb);
     }
-    for (int c = lh; c < vch; c += 4) cp_async_16(smem_u32(vd + c * 8), vsrc + (nb ? c * 8 : 0), nb);
+    for (int c = lh; c < vch; c += TPK) cp_async_16(smem_u32(vd + c * 8), vsrc + (nb ? c * 8 : 0), nb);
     cp_async_commit();
   };
   // Few rows (single tokens: at most 16 (token, head) pairs): all warps work on the SAME 16 rows, warp w on the keys
   // [16 (w & 3), +16) of every tile and half (w >> 2) of the value columns; the four partial softmaxes are merged at the end.
   // Otherwise warp w owns rows [16 w, +16) and walks whole tiles (warps without rows only help with the copies).
-  const bool few = ntok * group <= 16;
+  const bool few = WARPS == 8 && ntok * group <= 16;
   const int rbase = few ? 0 : warp * 16, kq = warp & 3, vh = warp >> 2;
   int pos[2], lo[2]; float qscale[2]; bool valid[2];
   const float* bias[2] = {nullptr, nullptr};
@@ -959,16 +961,19 @@ __global__ void __launch_bounds__(kThreads, DMAX > 128 ? 1 : 2) capped_attn_mma_
   }
 }
 
-template <int DMAX, int VMAX, int EXT>
+// WARPS 8: two CTAs per SM; 16: one CTA of twice the rows, for heads whose tiles are too large for two (every key tile is then
+// read by 256 rows instead of 128).
+template <int DMAX, int VMAX, int EXT, int WARPS = 8>
 int launch_mma(AttnArgs a, const int32_t* cu_tokens, int n_seqs, cudaStream_t st) {
+  constexpr int kRows = 16 * WARPS, kThreads = 32 * WARPS;
   const int group = a.heads / a.kv_heads, tq = kRows / group;
   const size_t tiles = (static_cast<size_t>(kRows) * (DMAX + 8) + 2 * kKeys * (DMAX + 8) + 2 * kKeys * (VMAX + 8)) * sizeof(bf16);
   const size_t bias_bytes = static_cast<size_t>(group) * a.dist_rows * sizeof(float);
   a.bias_staged = EXT == kExtTable && a.dist_bias != nullptr && bias_bytes <= kBiasSmemBytes;
   const size_t smem = tiles + (a.bias_staged ? bias_bytes : 0);
-  NVLLM_SMEM_ATTR_ONCE((capped_attn_mma_kernel<DMAX, VMAX, EXT>), tiles + (EXT == kExtTable ? kBiasSmemBytes : 0));
+  NVLLM_SMEM_ATTR_ONCE((capped_attn_mma_kernel<DMAX, VMAX, EXT, WARPS>), tiles + (EXT == kExtTable ? kBiasSmemBytes : 0));
   dim3 grid((a.n + tq - 1) / tq + n_seqs, a.kv_heads);
-  capped_attn_mma_kernel<DMAX, VMAX, EXT><<<grid, kThreads, smem, st>>>(a, cu_tokens, n_seqs, tq, group);
+  capped_attn_mma_kernel<DMAX, VMAX, EXT, WARPS><<<grid, kThreads, smem, st>>>(a, cu_tokens, n_seqs, tq, group);
   NVLLM_LAUNCH_CHECK("capped_attn_mma_kernel");
   return 0;
 }
@@ -1211,7 +1216,7 @@ extern "C" int nvllm_extended_attention(void* out, int64_t ldo, const void* q, i
   if (dim <= 64 && vdim <= 64) return launch_mma<64, 64, EXTV>(a, cu_tokens, n_seqs, st);             \
   if (vdim <= 64) return launch_mma<128, 64, EXTV>(a, cu_tokens, n_seqs, st);                         \
   return launch_mma<128, 128, EXTV>(a, cu_tokens, n_seqs, st)
-      if (dim > 128) return launch_mma<192, 128, kExtNone>(a, cu_tokens, n_seqs, st);
+      if (dim > 128) return launch_mma<192, 128, kExtNone, 16>(a, cu_tokens, n_seqs, st);
       if (ext == kExtNone) { NVLLM_ATTN(kExtNone); }
       if (ext == kExtSlope) { NVLLM_ATTN(kExtSlope); }
       NVLLM_ATTN(kExtTable);

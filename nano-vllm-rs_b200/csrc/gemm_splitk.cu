@@ -73,10 +73,11 @@ __device__ __forceinline__ void st_smem_f32(uint32_t addr, float v) {
 
 // One cluster of SK CTAs per (m_tile, n_tile); cluster rank r accumulates k-blocks [r * kb_per, (r + 1) * kb_per).
 // GATE: w = [gate (N rows) | up (N rows)], the B tile is BN/2 gate rows + the matching BN/2 up rows, y[:, BN/2 per tile].
-template <int BN, int SK, int GATE>
+template <int BN, int SK, int GATE, typename OutT>
 __global__ void __launch_bounds__(256, 1)
 gemm_splitk_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_constant__ CUtensorMap tmap_w,
-                   bf16* __restrict__ y, int M, int N, int K, int64_t ldy, int num_m_tiles, int STAGES, const RowPush ps, float glu_limit) {
+                   OutT* __restrict__ y, int M, int N, int K, int64_t ldy, int num_m_tiles, int STAGES, const RowPush ps, float glu_limit) {
+  static_assert(sizeof(OutT) == 2 || GATE == kGateNone, "the gated form writes bf16");
   using C = SkCfg<BN>;
   extern __shared__ uint8_t smem_raw[];
   const uint32_t smem_base = (smem_u32(smem_raw) + 1023u) & ~1023u;
@@ -198,7 +199,7 @@ gemm_splitk_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_cons
     if constexpr (GATE != kGateNone) {
       constexpr int CW = BN / (2 * SK);  // output columns of this CTA
       static_assert(CW >= 8 && CW % 8 == 0, "slice must be whole 16-byte vectors");
-      bf16* dst = y + row * ldy + n_tile * (BN / 2) + rank * CW;
+      bf16* dst = reinterpret_cast<bf16*>(y) + row * ldy + n_tile * (BN / 2) + rank * CW;
 #pragma unroll 1
       for (int j = 0; j < CW; j += 8) {
         const int cg = rank * CW + j, cu = BN / 2 + cg;
@@ -232,10 +233,12 @@ gemm_splitk_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_cons
       constexpr int CW = BN / SK;
       static_assert(CW >= 8 && CW % 8 == 0, "slice must be whole 16-byte vectors");
       constexpr int CH = (CW % 16 == 0 && SK <= 4) ? 16 : 8;  // columns per iteration: CH * SK coalesced loads in flight
-      bf16* dst = y + row * ldy + n_tile * BN + rank * CW;
+      OutT* dst = y + row * ldy + n_tile * BN + rank * CW;
       bool remote = false;  // TP: the row is reduced by another rank -> straight into its low-latency stage buffer
-      if (ps.ctrl != nullptr && row < M) {
-        if (bf16* pr = push_row(ps, row)) { dst = pr + n_tile * BN + rank * CW; remote = true; }
+      if constexpr (sizeof(OutT) == 2) {
+        if (ps.ctrl != nullptr && row < M) {
+          if (bf16* pr = push_row(ps, row)) { dst = pr + n_tile * BN + rank * CW; remote = true; }
+        }
       }
 #pragma unroll 1
       for (int j = 0; j < CW; j += CH) {
@@ -256,9 +259,14 @@ gemm_splitk_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_cons
         if (row < M) {
 #pragma unroll
           for (int e = 0; e < CH; e += 8) {
+            if constexpr (sizeof(OutT) == 4) {
+              reinterpret_cast<float4*>(dst + j + e)[0] = make_float4(a[e], a[e + 1], a[e + 2], a[e + 3]);
+              reinterpret_cast<float4*>(dst + j + e)[1] = make_float4(a[e + 4], a[e + 5], a[e + 6], a[e + 7]);
+              continue;
+            }
             const uint4 o = make_uint4(pack_bf16x2(a[e], a[e + 1]), pack_bf16x2(a[e + 2], a[e + 3]),
                                        pack_bf16x2(a[e + 4], a[e + 5]), pack_bf16x2(a[e + 6], a[e + 7]));
-            if (remote) st_sys_16(dst + j + e, ll_scrub(o));
+            if (remote) st_sys_16(reinterpret_cast<bf16*>(dst) + j + e, ll_scrub(o));
             else *reinterpret_cast<uint4*>(dst + j + e) = o;
           }
         }
@@ -300,11 +308,11 @@ int splitk_stages(int kb_per) {
   return want < kb_per ? want : (kb_per < 1 ? 1 : kb_per);
 }
 
-template <int BN, int SK, int GATE>
+template <int BN, int SK, int GATE, typename OutT = bf16>
 int launch_splitk(const CUtensorMap& tx, const CUtensorMap& tw, void* y, int M, int N, int K, int64_t ldy, int tiles,
                   int num_m_tiles, cudaStream_t st, const RowPush& ps, float glu_limit = 0.f) {
   using C = SkCfg<BN>;
-  auto kern = gemm_splitk_kernel<BN, SK, GATE>;
+  auto kern = gemm_splitk_kernel<BN, SK, GATE, OutT>;
   NVLLM_SMEM_ATTR_ONCE(kern, C::smem_bytes(C::kMaxStages));
   const int stages = splitk_stages<BN>((K / C::BK) / SK);
   cudaLaunchConfig_t cfg{};
@@ -319,7 +327,7 @@ int launch_splitk(const CUtensorMap& tx, const CUtensorMap& tw, void* y, int M, 
   attr[1].val.programmaticStreamSerializationAllowed = 1;
   cfg.attrs = attr;
   cfg.numAttrs = pdl_enabled() ? 2 : 1;
-  NVLLM_CUDA(cudaLaunchKernelEx(&cfg, kern, tx, tw, static_cast<bf16*>(y), M, N, K, ldy, num_m_tiles, stages, ps, glu_limit));
+  NVLLM_CUDA(cudaLaunchKernelEx(&cfg, kern, tx, tw, static_cast<OutT*>(y), M, N, K, ldy, num_m_tiles, stages, ps, glu_limit));
   return 0;
 }
 
@@ -346,6 +354,7 @@ bool splitk_choose(int m, int n_acc, int k, bool silu, int bn_default, int* out_
   auto legal = [&](int bn, int sk) {
     if (n_acc % bn != 0 || num_kb % sk != 0 || num_kb / sk < 1) return false;
     if ((silu ? bn / (2 * sk) : bn / sk) < 8 || (bn == 64 && sk == 8)) return false;
+    if (bn == 32 && (silu || n_acc % 64 == 0)) return false;   // only where no wider tile divides the columns
     return static_cast<long>(mt) * (n_acc / bn) * sk <= sms;
   };
   if (kn.splitk_mode == 2) {
@@ -354,7 +363,7 @@ bool splitk_choose(int m, int n_acc, int k, bool silu, int bn_default, int* out_
     if (known && legal(fbn, fsk)) { *out_bn = fbn; *out_sk = fsk; return true; }
     return false;
   }
-  const int bns[3] = {256, 128, 64}, sks[3] = {8, 4, 2};
+  const int bns[4] = {256, 128, 64, 32}, sks[3] = {8, 4, 2};
   long best = -1;
   for (int bn : bns)
     for (int sk : sks) {
@@ -381,7 +390,7 @@ namespace nvllm {
 #endif
 
 int gemm_splitk_dispatch(void* y, const void* x, const void* w, int m, int n, int k, int64_t ldx, int64_t ldw, int64_t ldy,
-                         int gate, int bn, int sk, cudaStream_t st, const RowPush& ps, float glu_limit) {
+                         int gate, int bn, int sk, cudaStream_t st, const RowPush& ps, float glu_limit, int out_dtype) {
   CUtensorMap tx, tw;
   const bool gated = gate != kGateNone;
   const int n_acc = gated ? 2 * n : n;
@@ -390,7 +399,8 @@ int gemm_splitk_dispatch(void* y, const void* x, const void* w, int m, int n, in
   const int mt = (m + 127) / 128, tiles = mt * (n_acc / bn);
 #define NVLLM_SK(BNV, SKV)                                                                                   \
   if (bn == BNV && sk == SKV)                                                                                \
-    return !gated                 ? launch_splitk<BNV, SKV, kGateNone>(tx, tw, y, m, n, k, ldy, tiles, mt, st, ps)                       \
+    return out_dtype == NVLLM_F32 ? launch_splitk<BNV, SKV, kGateNone, float>(tx, tw, y, m, n, k, ldy, tiles, mt, st, RowPush{})        \
+           : !gated               ? launch_splitk<BNV, SKV, kGateNone>(tx, tw, y, m, n, k, ldy, tiles, mt, st, ps)                       \
            : gate == kGateClamped ? launch_splitk<BNV, SKV, kGateClamped>(tx, tw, y, m, n, k, ldy, tiles, mt, st, RowPush{}, glu_limit) \
            : gate == kGateGelu    ? launch_splitk<BNV, SKV, kGateGelu>(tx, tw, y, m, n, k, ldy, tiles, mt, st, RowPush{})               \
                                   : launch_splitk<BNV, SKV, kGateSilu>(tx, tw, y, m, n, k, ldy, tiles, mt, st, RowPush{})
@@ -398,6 +408,12 @@ int gemm_splitk_dispatch(void* y, const void* x, const void* w, int m, int n, in
   NVLLM_SK(128, 8); NVLLM_SK(128, 4); NVLLM_SK(128, 2);
   NVLLM_SK(64, 4); NVLLM_SK(64, 2);
 #undef NVLLM_SK
+#define NVLLM_SK32(SKV)   /* narrow outputs (routers): no gated form */                                              \
+  if (bn == 32 && sk == SKV && !gated)                                                                              \
+    return out_dtype == NVLLM_F32 ? launch_splitk<32, SKV, kGateNone, float>(tx, tw, y, m, n, k, ldy, tiles, mt, st, RowPush{}) \
+                                  : launch_splitk<32, SKV, kGateNone>(tx, tw, y, m, n, k, ldy, tiles, mt, st, ps)
+  NVLLM_SK32(4); NVLLM_SK32(2);
+#undef NVLLM_SK32
   NVLLM_CHECK_ARG(false, NVLLM_ERR_ARG, "gemm_splitk: no kernel for bn=%d sk=%d", bn, sk);
 }
 

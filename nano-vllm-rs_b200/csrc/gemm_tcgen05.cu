@@ -442,7 +442,7 @@ int gemm_silu_2cta_dispatch(void* y, const void* x, const void* w, int m, int in
 // gemm_splitk.cu: cluster split-K for decode-sized projections (m <= 256)
 bool splitk_choose(int m, int n_acc, int k, bool silu, int bn_default, int* out_bn, int* out_sk);
 int gemm_splitk_dispatch(void* y, const void* x, const void* w, int m, int n, int k, int64_t ldx, int64_t ldw, int64_t ldy,
-                         int gate, int bn, int sk, cudaStream_t st, const RowPush& ps = RowPush{}, float glu_limit = 0.f);
+                         int gate, int bn, int sk, cudaStream_t st, const RowPush& ps = RowPush{}, float glu_limit = 0.f, int out_dtype = NVLLM_BF16);
 
 static bool use_2cta();
 // CTA pairs pay off once there are at least two 256-row tiles or the problem is large enough to fill the machine with
@@ -488,10 +488,10 @@ int gemm_bf16_impl(void* y, const void* x, const void* w, int32_t m, int32_t n, 
   if (m == 0) return 0;
   NVLLM_CHECK_ARG(y && x && w && aligned16(y) && aligned16(x) && aligned16(w), NVLLM_ERR_ALIGN, "gemm: pointers");
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (out_dtype == NVLLM_BF16) {  // decode-sized, long-K projections: split K over a cluster (gemm_splitk.cu)
+  {  // decode-sized, long-K projections: split K over a cluster (gemm_splitk.cu)
     int sbn = 0, ssk = 0;
     if (splitk_choose(m, n, k, false, pick_bn(m, n), &sbn, &ssk))
-      return gemm_splitk_dispatch(y, x, w, m, n, k, ldx, ldw, ldy, kGateNone, sbn, ssk, st, ps);
+      return gemm_splitk_dispatch(y, x, w, m, n, k, ldx, ldw, ldy, kGateNone, sbn, ssk, st, ps, 0.f, out_dtype);
   }
   if (!push && want_2cta(m, n, k)) return gemm_2cta_dispatch(y, x, w, m, n, k, ldx, ldw, ldy, out_dtype, st);
   const int bn = pick_bn(m, n);

@@ -759,3 +759,148 @@ def gemm_glu_grouped(x, w, tile_group, inter, groups, limit):
     check(_ffi.lib().nvllm_gemm_glu_bf16_grouped(_p(out), _p(x), _p(w), rows, inter, K, groups, x.stride(0), w.stride(0), out.stride(0),
                                                  _p(tile_group), limit, _stream()))
     return out
+
+
+# ---- capped scores with a slope per head, keys in two parts, YaRN, element-wise output gates, gelu gates, experts that scale their input
+
+
+def extended_attention(q, gate, k_cache, v_cache, tok_seq, positions, tables, block_size, heads, kv_heads, dim, vdim, scale, softcap=0.0, temp_coef=0.0,
+                       temp_every=1, window=0, slopes=None, k_shared=None, shared_dim=0, cu_tokens=None):
+    """Attention with a cap, a query temperature, a slope per head taken off by distance, and keys whose last shared_dim values are
+    the rows of k_shared (one per cache slot).  tables None: dense rows, key j of sequence s is row cu_tokens[s] + j."""
+    n = q.shape[0]
+    out = torch.empty((n, heads * vdim), dtype=q.dtype, device=q.device)
+    check(_ffi.lib().nvllm_extended_attention(_p(out), out.stride(0), _p(q), q.stride(0), _p(gate), gate.stride(0) if gate is not None else 0, 0,
+                                              _p(k_cache), _p(v_cache), k_cache.stride(0), v_cache.stride(0), _p(tok_seq), _p(positions), _p(tables),
+                                              tables.shape[1] if tables is not None else 1, block_size, n, heads, kv_heads, dim, vdim, scale, softcap,
+                                              temp_coef, temp_every, window, 0, None, 0, None, None, 0, None, 0, _p(slopes), _p(k_shared),
+                                              k_shared.stride(0) if k_shared is not None else 0, shared_dim, _p(cu_tokens),
+                                              cu_tokens.shape[0] - 1 if cu_tokens is not None else 0, _dt(q), _stream()))
+    return out
+
+
+def attn_store(proj, q_cols, k_cols, v_cols, k_cache, v_cache, slots, dtype):
+    """Columns [q | k | v] of proj (f32): q returned in `dtype`, k and v into cache rows `slots`."""
+    n = proj.shape[0]
+    q = torch.empty((n, q_cols), dtype=dtype, device=proj.device)
+    check(_ffi.lib().nvllm_attn_bias_store(_p(q), q.stride(0), _p(k_cache), _p(v_cache), k_cache.stride(0), v_cache.stride(0), _p(proj), proj.stride(0),
+                                           None, None, None, _p(slots), n, q_cols, k_cols, v_cols, _dt(q), _stream()))
+    return q
+
+
+def rope_table_yarn(max_pos, dims, base, factor, fast, slow, original, device):
+    """[max_pos, dims / 2, 2] of (cos, sin) with YaRN frequencies and amplitude."""
+    tab = torch.empty((max_pos, dims // 2, 2), dtype=torch.float32, device=device)
+    check(_ffi.lib().nvllm_rope_table_yarn(_p(tab), max_pos, dims, float(base), float(factor), float(fast), float(slow), float(original), _stream()))
+    return tab
+
+
+def latent_norm_store(proj, q_rank, dq_norm_w, kv_off, kv_rank, rot_dim, c_norm_w, eps, positions, table, rot_dims, cache, slots, dtype, dense=None):
+    """Returns rms(proj[:, :q_rank]) * dq_norm_w; [rms(latent) * c_norm_w | rotated key part] goes to cache rows `slots` (and `dense`)."""
+    n = proj.shape[0]
+    cq = torch.empty((n, q_rank), dtype=dtype, device=proj.device)
+    check(_ffi.lib().nvllm_latent_norm_store(_p(cq), cq.stride(0), _p(proj), proj.stride(0), q_rank, _p(dq_norm_w), kv_off, kv_rank, rot_dim, _p(c_norm_w),
+                                             eps, _p(positions), _p(table), rot_dims, table.shape[0] if table is not None else 1, _p(cache), _p(dense),
+                                             cache.stride(0), _p(slots), n, _dt(cq), _stream()))
+    return cq
+
+
+def rotate_tail(x, positions, table, rot_dims, heads, dim, rot_dim):
+    """In place: the first rot_dims of every head's last rot_dim values are rotated (neighbouring pairs)."""
+    check(_ffi.lib().nvllm_rotate_tail(_p(x), x.stride(0), _p(positions), _p(table), rot_dims, table.shape[0] if table is not None else 1, x.shape[0],
+                                       heads, dim, rot_dim, _dt(x), _stream()))
+
+
+def latent_rotary_attention(q_abs, q, tok_seq, positions, tables, block_size, cache, heads, dim, rot_dim, kv_rank, scale, window=0, workspace=None):
+    """latent_window_attention whose cache rows also hold a rotated key part; q [n, heads * (dim + rot_dim)]."""
+    n = q_abs.shape[0]
+    out = torch.empty((n, heads * kv_rank), dtype=q.dtype, device=q_abs.device)
+    check(_ffi.lib().nvllm_latent_window_attention(_p(out), out.stride(0), _p(q_abs), q_abs.stride(0), _p(q), q.stride(0), _p(tok_seq), _p(positions),
+                                                   _p(tables), tables.shape[1], block_size, _p(cache), cache.stride(0), n, heads, dim, rot_dim, kv_rank,
+                                                   scale, window, None, None, 0, _p(workspace), workspace.numel() * 4 if workspace is not None else 0,
+                                                   _dt(out), _stream()))
+    return out
+
+
+def linear_gated(x, w, gate, batch, n, k, bsx, bsw, bsg, ldw=None):
+    """y[:, b n : (b + 1) n] = (x_b w_b^T) * sigmoid(gate_b): x [m, ldx] with heads bsx apart, w heads bsw apart, gate columns bsg apart."""
+    m = x.shape[0]
+    out = torch.empty((m, n * batch), dtype=x.dtype, device=x.device)
+    check(_ffi.lib().nvllm_linear_gated(_p(out), _p(x), _p(w), m, n, k, x.stride(0), ldw or k, out.stride(0), batch, bsx, bsw, n, _p(gate),
+                                        gate.stride(0) if gate is not None else 0, bsg, _dt(x), _dt(out), _stream()))
+    return out
+
+
+def sigmoid_gate(y, gate):
+    """y *= sigmoid(gate) in place; gate f32."""
+    check(_ffi.lib().nvllm_sigmoid_gate(_p(y), y.stride(0), _p(gate), gate.stride(0), y.shape[0], y.shape[1], _dt(y), _stream()))
+
+
+def token_gate(gate, table, col0, ids):
+    """gelu_tanh(gate) * table[ids, col0 : col0 + dim] in the table's type; gate f32 [n, >= dim columns of a view]."""
+    n, dim = gate.shape
+    out = torch.empty((n, dim), dtype=table.dtype, device=gate.device)
+    check(_ffi.lib().nvllm_token_gate(_p(out), _p(gate), gate.stride(0), _p(table), table.stride(0), col0, _p(ids), table.shape[0], n, dim, _dt(table),
+                                      _stream()))
+    return out
+
+
+GATES = {"silu": 1, "clamped": 2, "gelu": 3}
+
+
+def gated_gelu(gate_up):
+    """gelu_tanh of the first half of the columns times the second half."""
+    n, ff2 = gate_up.shape
+    out = torch.empty((n, ff2 // 2), dtype=gate_up.dtype, device=gate_up.device)
+    check(_ffi.lib().nvllm_ff_activation_params(_p(out), _p(gate_up), n, ff2 // 2, 3, None, _dt(gate_up), _stream()))
+    return out
+
+
+def gemm_gated(x, w_gate_up, gate, limit=0.0):
+    """gemm_glu with the gate named: "silu", "clamped" (limit) or "gelu"."""
+    _need(x, torch.bfloat16, "x"); _need(w_gate_up, torch.bfloat16, "w_gate_up")
+    M, K = x.shape
+    inter = w_gate_up.shape[0] // 2
+    out = torch.empty((M, inter), dtype=torch.bfloat16, device=x.device)
+    ws = torch.empty((M, 2 * inter), dtype=torch.bfloat16, device=x.device)
+    check(_ffi.lib().nvllm_gemm_gated_bf16(_p(out), _p(x), _p(w_gate_up), M, inter, K, x.stride(0), w_gate_up.stride(0), out.stride(0), GATES[gate], limit,
+                                           _p(ws), ws.numel() * 2, _stream()))
+    return out
+
+
+def gemm_gated_grouped(x, w, tile_group, inter, groups, gate, limit=0.0, row_scale=None):
+    """gemm_gated over 128-row expert tiles; row_scale (f32 [rows], SiLU only): a factor on every row of x."""
+    rows, K = x.shape
+    out = torch.empty((rows, inter), dtype=torch.bfloat16, device=x.device)
+    check(_ffi.lib().nvllm_gemm_gated_bf16_grouped(_p(out), _p(x), _p(w), rows, inter, K, groups, x.stride(0), w.stride(0), out.stride(0), _p(tile_group),
+                                                   GATES[gate], limit, _p(row_scale), _stream()))
+    return out
+
+
+def linear_grouped_scaled(x, w, row_src, row_scale, tile_group, max_rows, n, k, group_stride_w, glu=0, limit=0.0):
+    """linear_grouped with a factor per row on its input."""
+    out = torch.zeros((max_rows, n), dtype=x.dtype, device=x.device)
+    check(_ffi.lib().nvllm_linear_grouped_scaled(_p(out), _p(x), _p(w), max_rows, n, k, x.stride(0), k, n, group_stride_w, _p(row_src), _p(row_scale),
+                                                 _p(tile_group), int(glu), limit, _dt(x), _dt(x), _stream()))
+    return out
+
+
+def moe_route_sigmoid(logits, bias, top):
+    """The `top` largest of logits + bias (ties: lowest index) and their sigmoids, as they are."""
+    n, experts = logits.shape
+    idx = torch.empty((n, top), dtype=torch.int32, device=logits.device)
+    w = torch.empty((n, top), dtype=torch.float32, device=logits.device)
+    check(_ffi.lib().nvllm_moe_route_sigmoid(_p(idx), _p(w), _p(logits), logits.stride(0), _p(bias), n, experts, top, _stream()))
+    return idx, w
+
+
+def moe_sort_weighted(topk_idx, topk_w, experts, tile_rows=32):
+    """moe_sort that also returns every row's assignment weight (0 on padding rows)."""
+    n, top = topk_idx.shape
+    rows = _ffi.lib().nvllm_moe_max_rows(n, top, experts, tile_rows)
+    dev = topk_idx.device
+    row_token, row_w = torch.empty(rows, dtype=torch.int32, device=dev), torch.empty(rows, dtype=torch.float32, device=dev)
+    tile_expert, slot_row = torch.empty(rows // tile_rows, dtype=torch.int32, device=dev), torch.empty((n, top), dtype=torch.int32, device=dev)
+    check(_ffi.lib().nvllm_moe_sort_weighted(_p(row_token), _p(row_w), _p(tile_expert), _p(slot_row), _p(topk_idx), _p(topk_w), n, top, experts, rows,
+                                             tile_rows, _stream()))
+    return row_token, row_w, tile_expert, slot_row
