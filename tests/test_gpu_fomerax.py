@@ -336,6 +336,14 @@ def test_folded_latent_attention_with_a_rotated_part(cuda, dtype, H, R, rd, size
     assert np.abs(got - ref).max() < (2e-5 if dtype == F32 else 2e-2) * max(1.0, np.abs(ref).max()), np.abs(got - ref).max()
 
 
+def test_long_windows_share_their_keys_over_ctas(cuda):
+    """Single tokens in a window of more than a thousand keys: with a workspace their key tiles are split over several CTAs."""
+    for H, R, rd, size in ((6, 64, 32, 1200), (3, 128, 8, 2100)):
+        ws = torch.zeros(4 * 4 * H * (R + 2), device=cuda)
+        got, ref, _ = folded(cuda, np.random.default_rng(R), BF16, H, R, rd, size, [(1500, 1), (2300, 1), (90, 1), (0, 1)], 1.5 / np.sqrt(R + rd), workspace=ws)
+        assert np.abs(got - ref).max() < 2e-2 * max(1.0, np.abs(ref).max()), np.abs(got - ref).max()
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("portion", [1, 2, 40, 300])
 @pytest.mark.parametrize("size,bs,p", [(41, 64, 420), (64, 16, 383), (63, 16, 384), (33, 32, 351), (1, 16, 340), (128, 16, 511), (5, 16, 303)])
